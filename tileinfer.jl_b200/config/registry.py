@@ -14,6 +14,7 @@ from typing import Any, Callable, Dict, Mapping, Optional
 
 from .apertus import ApertusConfig, ConfigError
 from .fasodra import FasodraConfig
+from .midisun import MidisunConfig
 from .vogilix import VogilixConfig
 from .sozanex import SozanexConfig
 from .zudepel import ZudepelConfig
@@ -77,3 +78,4 @@ register_architecture(VogilixConfig.architecture, VogilixConfig, model_type=Vogi
 register_architecture(ZudepelConfig.architecture, ZudepelConfig, model_type=ZudepelConfig.model_type)
 register_architecture(SozanexConfig.architecture, SozanexConfig, model_type=SozanexConfig.model_type)
 register_architecture(FasodraConfig.architecture, FasodraConfig, model_type=FasodraConfig.model_type)
+register_architecture(MidisunConfig.architecture, MidisunConfig, model_type=MidisunConfig.model_type)

@@ -121,6 +121,8 @@ __global__ void __launch_bounds__(AD_THREADS) attention_decode_kernel(
     const int head0 = kvh * full_group + slab * 16;
     const float* bias0 = ex.bias != nullptr ? ex.bias + (size_t)(head0 + (g < group ? g : 0)) * ex.bias_len : nullptr;
     const float* bias1 = ex.bias != nullptr ? ex.bias + (size_t)(head0 + (g + 8 < group ? g + 8 : 0)) * ex.bias_len : nullptr;
+    const float slope0 = ex.slope != nullptr ? ex.slope[head0 + (g < group ? g : 0)] : 0.f;
+    const float slope1 = ex.slope != nullptr ? ex.slope[head0 + (g + 8 < group ? g + 8 : 0)] : 0.f;
 
     for (int tile = my_lo; tile < my_hi; ++tile) {
         const int stage = (tile - my_lo) % SM::STAGES;
@@ -131,7 +133,8 @@ __global__ void __launch_bounds__(AD_THREADS) attention_decode_kernel(
         const bf16* kt = tiles + (size_t)stage * 2 * SM::TILE;
         const bf16* vt = kt + SM::TILE;
 
-        decode_tile<D>(kt, vt, qf, o, m0, m1, l0, l1, tile, warp, lane, kv_len, first_key, scale_log2e, bias0, bias1, ex.bias_len);
+        decode_tile<D>(kt, vt, qf, o, m0, m1, l0, l1, tile, warp, lane, kv_len, first_key, scale_log2e, bias0, bias1, ex.bias_len, ex,
+                       slope0, slope1);
     }
     cp_async_wait<0>();
     __syncthreads();
@@ -275,15 +278,15 @@ static int launch_decode(bf16* out, const bf16* q, const bf16* k, const bf16* v,
 // part << 8 | parts (at most 32), or -1 for a slot left without work; the sequence's length), 8-byte aligned
 // pairs; seq_work[sequence] = first slot << 8 | parts; a sequence's slots are consecutive. Without them every sequence takes `splits` equal parts.
 // `sink` [nq] float (or null): one more term exp(sink[head]) in every softmax's denominator, with no key and no value.
-// `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`: see AttnExtras.
-extern "C" int ti_attention_decode_biased(void* out, const void* q, const void* k_cache, const void* v_cache,
+// `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`, `cap`, `slope` [nq] (times log2 e): see AttnExtras.
+extern "C" int ti_attention_decode_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
                                           const int* block_table, int table_stride, const int* seq_slots, const int* kv_lens,
                                           const int* work, const int* seq_work, float* ws_o, float* ws_ml, float scale, int B,
                                           int nq, int nkv, int D, int page_size, int splits, int window, const float* sink, int chunk,
-                                          const float* dist_bias, int bias_len, cudaStream_t stream) {
+                                          const float* dist_bias, int bias_len, float cap, const float* slope, cudaStream_t stream) {
     if (B == 0) return 0;
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention_decode: chunk %d, bias table of %d", chunk, bias_len);
-    const AttnExtras ex = {chunk, dist_bias, bias_len};
+    const AttnExtras ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope);
     if (page_size != AD_PAGE || nq % nkv != 0 || nq / nkv > 128 || D % 16 != 0 || B > 32767 || (long long)nkv * ((nq / nkv + 15) / 16) > 65535) {
         ti_fail("attention_decode takes page size %d, at most 128 query heads per KV head and head sizes in steps of 16; "
                 "got page %d, %d/%d heads, head size %d", AD_PAGE, page_size, nq, nkv, D);
@@ -304,6 +307,15 @@ extern "C" int ti_attention_decode_biased(void* out, const void* q, const void* 
             return 2;
     }
 #undef AD_CASE
+}
+
+extern "C" int ti_attention_decode_biased(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                          const int* block_table, int table_stride, const int* seq_slots, const int* kv_lens,
+                                          const int* work, const int* seq_work, float* ws_o, float* ws_ml, float scale, int B,
+                                          int nq, int nkv, int D, int page_size, int splits, int window, const float* sink, int chunk,
+                                          const float* dist_bias, int bias_len, cudaStream_t stream) {
+    return ti_attention_decode_ruled(out, q, k_cache, v_cache, block_table, table_stride, seq_slots, kv_lens, work, seq_work, ws_o, ws_ml, scale,
+                                     B, nq, nkv, D, page_size, splits, window, sink, chunk, dist_bias, bias_len, 0.f, nullptr, stream);
 }
 
 extern "C" int ti_attention_decode_sink(void* out, const void* q, const void* k_cache, const void* v_cache,

@@ -29,7 +29,8 @@ __global__ void attention_plain_kernel(T* __restrict__ out, const T* q, const T*
                                        int table_stride, const int* tok_slot,
                                        const int* positions, float scale, int nq, int nkv, int D,
                                        int page_size, int window, const float* __restrict__ sink, int chunk,
-                                       const float* __restrict__ dist_bias, int bias_len) {
+                                       const float* __restrict__ dist_bias, int bias_len, float cap,
+                                       const float* __restrict__ slope) {
     extern __shared__ float smem[];
     float* qs = smem;                          // [AP_HEADS][D]
     float* sc = smem + AP_HEADS * D;           // [AP_HEADS][AP_CHUNK]
@@ -95,8 +96,10 @@ __global__ void attention_plain_kernel(T* __restrict__ out, const T* q, const T*
             for (int h = 0; h < AP_HEADS; ++h)
                 if (h < heads) {
                     s[h] *= scale;
+                    if (cap > 0.f) s[h] = cap * tanhf(s[h] / cap);
                     // A learned bias per (head, distance), added after the scale; distances beyond the table take its last entry.
                     if (dist_bias != nullptr) s[h] += dist_bias[(size_t)(h0 + h) * bias_len + min(p - j, bias_len - 1)];
+                    if (slope != nullptr) s[h] = fmaf(-slope[h0 + h], (float)(p - j), s[h]);
                     sc[h * AP_CHUNK + j - c0] = s[h];
                     cmax[h] = fmaxf(cmax[h], s[h]);
                 }
@@ -153,11 +156,13 @@ __global__ void attention_plain_kernel(T* __restrict__ out, const T* q, const T*
 }
 
 // `chunk` > 0: a key is visible only inside the query's chunk of so many positions; `dist_bias` [nq][bias_len] float: added to
-// the scaled score by the distance between query and key (null: none).
-extern "C" int ti_attention_plain_biased(void* out, const void* q, const void* k_cache, const void* v_cache,
-                                         const int* block_table, int table_stride, const int* tok_slot, const int* positions,
+// the scaled score by the distance between query and key (null: none). `cap` > 0: the scaled score s becomes cap tanh(s / cap) before
+// any bias; `slope` [nq] float (null: none): slope[head] * distance is taken off after the cap.
+extern "C" int ti_attention_plain_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                        const int* block_table, int table_stride, const int* tok_slot, const int* positions,
                                          float scale, int n_tokens, int nq, int nkv, int D, int page_size, int window,
-                                         const float* sink, int chunk, const float* dist_bias, int bias_len, int dtype, cudaStream_t stream) {
+                                         const float* sink, int chunk, const float* dist_bias, int bias_len, float cap, const float* slope,
+                                        int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention: chunk %d, bias table of %d", chunk, bias_len);
     TI_REQUIRE(D > 0 && D <= AP_MAX_D, "attention: head_dim %d exceeds %d", D, AP_MAX_D);
@@ -168,8 +173,16 @@ extern "C" int ti_attention_plain_biased(void* out, const void* q, const void* k
     const size_t smem = (size_t)AP_HEADS * (D + AP_CHUNK) * sizeof(float);
     TI_DISPATCH_DTYPE(dtype, (ti_launch(attention_plain_kernel<T>, dim3(grid), dim3(AP_THREADS), smem, stream, 
                                  (T*)out, (const T*)q, (const T*)k_cache, (const T*)v_cache, block_table, table_stride,
-                                 tok_slot, positions, scale, nq, nkv, D, page_size, window, sink, chunk, dist_bias, bias_len)));
+                                 tok_slot, positions, scale, nq, nkv, D, page_size, window, sink, chunk, dist_bias, bias_len, cap, slope)));
     return ti_check_launch("attention_plain");
+}
+
+extern "C" int ti_attention_plain_biased(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                         const int* block_table, int table_stride, const int* tok_slot, const int* positions,
+                                         float scale, int n_tokens, int nq, int nkv, int D, int page_size, int window,
+                                         const float* sink, int chunk, const float* dist_bias, int bias_len, int dtype, cudaStream_t stream) {
+    return ti_attention_plain_ruled(out, q, k_cache, v_cache, block_table, table_stride, tok_slot, positions, scale, n_tokens, nq, nkv, D,
+                                    page_size, window, sink, chunk, dist_bias, bias_len, 0.f, nullptr, dtype, stream);
 }
 
 extern "C" int ti_attention_plain(void* out, const void* q, const void* k_cache, const void* v_cache,

@@ -87,6 +87,8 @@ __global__ void __launch_bounds__(PF_THREADS, 1) attention_prefill_kernel(
     const int lo0 = first_seen(pos0), lo1 = first_seen(pos1);
     const float* bias0 = ex.bias != nullptr ? ex.bias + (size_t)(kvh * group + r0 % group) * ex.bias_len : nullptr;
     const float* bias1 = ex.bias != nullptr ? ex.bias + (size_t)(kvh * group + r1 % group) * ex.bias_len : nullptr;
+    const float slope0 = ex.slope != nullptr ? ex.slope[kvh * group + r0 % group] : 0.f;
+    const float slope1 = ex.slope != nullptr ? ex.slope[kvh * group + r1 % group] : 0.f;
 
     unsigned qf[KS][4];
     {
@@ -162,6 +164,11 @@ __global__ void __launch_bounds__(PF_THREADS, 1) attention_prefill_kernel(
             for (int j = 0; j < 2; ++j) {
                 const int key = key_base + 8 * nt + 2 * t + j;
                 float a = s[nt][j] * scale_log2e, c = s[nt][2 + j] * scale_log2e;
+                if (ex.cap_out > 0.f) { a = capped_score2(s[nt][j], ex); c = capped_score2(s[nt][2 + j], ex); }
+                if (ex.slope != nullptr) {                   // (rows that do not see the key are masked below)
+                    a = fmaf(slope0, (float)(key - pos0), a);
+                    c = fmaf(slope1, (float)(key - pos1), c);
+                }
                 if (bias0 != nullptr) {                      // the bias of the distance, per row's head; rows that do not see the key are masked below
                     a += bias0[min(max(pos0 - key, 0), ex.bias_len - 1)];
                     c += bias1[min(max(pos1 - key, 0), ex.bias_len - 1)];
@@ -251,13 +258,13 @@ static int launch_prefill(bf16* out, const bf16* q, const bf16* k, const bf16* v
 // tokens_per_tile = 128 / (query heads per KV head). Returns 2 when the sizes are outside what the
 // kernel takes (the caller then runs the plain kernel).
 // `sink` [nq] float (or null): one more term exp(sink[head]) in every softmax's denominator.
-// `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`: see AttnExtras.
-extern "C" int ti_attention_prefill_biased(void* out, const void* q, const void* k_cache, const void* v_cache,
+// `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`, `cap`, `slope` [nq] (times log2 e): see AttnExtras.
+extern "C" int ti_attention_prefill_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
                                          const int* block_table, int table_stride, const int* seq_slots,
                                          const int* cu_seqlens, const int* kv_lens, int n_seqs, int total_tiles, float scale,
                                          int nq, int nkv, int D, int page_size, int window, const float* sink, int chunk, const float* dist_bias, int bias_len,
-                                           cudaStream_t stream) {
-    const AttnExtras ex = {chunk, dist_bias, bias_len};
+                                         float cap, const float* slope, cudaStream_t stream) {
+    const AttnExtras ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope);
     if (n_seqs == 0 || total_tiles == 0) return 0;
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention_prefill: chunk %d, bias table of %d", chunk, bias_len);
     if (page_size != PF_PAGE || nq % nkv != 0 || nq / nkv > PF_ROWS || D % 16 != 0 || nkv > 65535) {
@@ -278,6 +285,15 @@ extern "C" int ti_attention_prefill_biased(void* out, const void* q, const void*
             return 2;
     }
 #undef PF_CASE
+}
+
+extern "C" int ti_attention_prefill_biased(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                           const int* block_table, int table_stride, const int* seq_slots,
+                                           const int* cu_seqlens, const int* kv_lens, int n_seqs, int total_tiles, float scale,
+                                           int nq, int nkv, int D, int page_size, int window, const float* sink, int chunk, const float* dist_bias,
+                                           int bias_len, cudaStream_t stream) {
+    return ti_attention_prefill_ruled(out, q, k_cache, v_cache, block_table, table_stride, seq_slots, cu_seqlens, kv_lens, n_seqs, total_tiles,
+                                      scale, nq, nkv, D, page_size, window, sink, chunk, dist_bias, bias_len, 0.f, nullptr, stream);
 }
 
 extern "C" int ti_attention_prefill_sink(void* out, const void* q, const void* k_cache, const void* v_cache,

@@ -247,7 +247,10 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
         const unsigned lane_base = tmem_base + ((unsigned)((warp & 3) * 32) << 16);
         const unsigned s_addr = lane_base + x * KEYS, o_addr = lane_base + C::O_COL + x * D;
         float m_used = -1e30f, l = 0.f;
-        const float score_scale = p.ex.bias != nullptr ? 1.0f : p.scale_log2;      // with a bias the scores are scaled where it is added
+        // With a cap, a bias or a slope the scores are in base-2 units from where that is applied on.
+        const bool shaped = p.ex.bias != nullptr || p.ex.cap_out > 0.f || p.ex.slope != nullptr;
+        const float score_scale = shaped ? 1.0f : p.scale_log2;
+        const float slope = p.ex.slope != nullptr ? __ldg(p.ex.slope + min(head, p.heads - 1)) : 0.f;
         bool ok = true;
         for (int j = j_lo; ok && j < j_hi; ++j) {
             const unsigned jphase = (unsigned)(j - j_lo) & 1u;
@@ -266,6 +269,17 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
 #pragma unroll
             for (int c = 0; c < 4; ++c) tmem_ld32(s_addr + c * 32, r[c]);
             tmem_ld_wait();
+            if (p.ex.cap_out > 0.f || p.ex.slope != nullptr) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) {
+                        const float raw = __uint_as_float(r[c][i]);
+                        const float s = p.ex.cap_out > 0.f ? capped_score2(raw, p.ex) : raw * p.scale_log2;
+                        r[c][i] = __float_as_uint(fmaf(slope, (float)(key0 + c * 32 + i - pos), s));
+                    }
+            }
+            const float bias_scale = p.ex.cap_out > 0.f || p.ex.slope != nullptr ? 1.0f : p.scale_log2;
             if (p.ex.bias != nullptr) {
                 // A bias by the distance to the key, added to the scaled score: from here on the scores are in base-2 units
                 // (the scale below is then one). Keys that the row does not see are masked afterwards.
@@ -275,7 +289,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         const int dist = min(max(pos - (key0 + c * 32 + i), 0), p.ex.bias_len - 1);
-                        r[c][i] = __float_as_uint(fmaf(__uint_as_float(r[c][i]), p.scale_log2, __ldg(brow + dist)));
+                        r[c][i] = __float_as_uint(fmaf(__uint_as_float(r[c][i]), bias_scale, __ldg(brow + dist)));
                     }
             }
             if (masked) {
@@ -404,12 +418,13 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 // non-zero value afterwards means a wait ran out. Returns 2 when the sizes are outside what this kernel
 // takes (head size 64 or 128, 1 to 128 query heads per KV head, pages of 64): the caller then runs the
 // kernel for all sizes.
-// `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`: see AttnExtras.
-extern "C" int ti_attention_prefill_tc_biased(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,
+// `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`, `cap`, `slope` [nq] (times log2 e): see AttnExtras.
+extern "C" int ti_attention_prefill_tc_ruled(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,
                                               const int* block_table, int table_stride, const int* seq_slots,
                                               const int* cu_seqlens, const int* kv_lens, int n_seqs, int n_tokens, int total_blocks,
                                               float scale, int nq, int nkv, int D, int page_size, int window, int* status,
-                                              const float* sink, int chunk, const float* dist_bias, int bias_len, cudaStream_t stream) {
+                                              const float* sink, int chunk, const float* dist_bias, int bias_len, float cap, const float* slope,
+                                             cudaStream_t stream) {
     if (n_seqs == 0 || total_blocks == 0) return 0;
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention_prefill_tc: chunk %d, bias table of %d", chunk, bias_len);
     const int group = nkv > 0 ? nq / nkv : 0;
@@ -424,7 +439,7 @@ extern "C" int ti_attention_prefill_tc_biased(void* out, const void* q, const vo
     p.out = (bf16*)out; p.table = block_table; p.table_stride = table_stride; p.slots = seq_slots; p.cu_seqlens = cu_seqlens;
     p.kv_lens = kv_lens; p.n_seqs = n_seqs; p.heads = nq; p.kv_heads = nkv; p.group = group; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.sink = sink;
-    p.ex = AttnExtras{chunk, dist_bias, bias_len};
+    p.ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope);
     CUtensorMap mq, mk, mv;
     {
         const unsigned long long dims[3] = {(unsigned long long)D, (unsigned long long)nq, (unsigned long long)n_tokens};
@@ -441,6 +456,16 @@ extern "C" int ti_attention_prefill_tc_biased(void* out, const void* q, const vo
     }
     return D == 64 ? launch<64>(mq, mk, mv, (const bf16*)q, p, total_blocks, stream)
                    : launch<128>(mq, mk, mv, (const bf16*)q, p, total_blocks, stream);
+}
+
+extern "C" int ti_attention_prefill_tc_biased(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,
+                                              const int* block_table, int table_stride, const int* seq_slots,
+                                              const int* cu_seqlens, const int* kv_lens, int n_seqs, int n_tokens, int total_blocks,
+                                              float scale, int nq, int nkv, int D, int page_size, int window, int* status,
+                                              const float* sink, int chunk, const float* dist_bias, int bias_len, cudaStream_t stream) {
+    return ti_attention_prefill_tc_ruled(out, q, k_cache, v_cache, n_pages, block_table, table_stride, seq_slots, cu_seqlens, kv_lens, n_seqs,
+                                         n_tokens, total_blocks, scale, nq, nkv, D, page_size, window, status, sink, chunk, dist_bias, bias_len,
+                                         0.f, nullptr, stream);
 }
 
 extern "C" int ti_attention_prefill_tc_sink(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,

@@ -216,12 +216,26 @@ __host__ __forceinline__ bool aligned16(const void* p) { return ((uintptr_t)p & 
 // Two more rules of visibility and score for the paged attention kernels. chunk > 0: a key is visible only inside the query's
 // chunk of so many positions, floor(i / chunk) = floor(j / chunk), counted from the sequence's start. bias [heads][bias_len]
 // (null: none): entry [head][min(i - j, bias_len - 1)] is added to the scaled score; the kernels that work in base 2 get the
-// table already times log2(e).
+// table already times log2(e). cap_out > 0: the scaled score s becomes cap * tanh(s / cap), before any bias; slope [heads] (null:
+// none): slope[head] * (i - j) is taken off afterwards. The kernels that work in base 2 read cap_in = 2 scale log2(e) / cap (it
+// multiplies the unscaled score), cap_out = cap log2(e) and slopes times log2(e).
 struct AttnExtras {
     int chunk;
     const float* bias;
     int bias_len;
+    float cap_in = 0.f, cap_out = 0.f;
+    const float* slope = nullptr;
 };
+inline AttnExtras attn_extras(int chunk, const float* bias, int bias_len, float scale, float cap, const float* slope) {
+    AttnExtras ex = {chunk, bias, bias_len};
+    if (cap > 0.f) { ex.cap_in = 2.f * scale * 1.4426950408889634f / cap; ex.cap_out = cap * 1.4426950408889634f; }
+    ex.slope = slope;
+    return ex;
+}
+// cap log2(e) tanh(scale * raw / cap) as cap_out (1 - 2 / (1 + 2^(cap_in raw))): its error is a rounding of cap_out, whatever the score.
+__device__ __forceinline__ float capped_score2(float raw, const AttnExtras& ex) {
+    return fmaf(-2.f * ex.cap_out, __fdividef(1.f, 1.f + exp2f(ex.cap_in * raw)), ex.cap_out);
+}
 
 #define TI_DISPATCH_DTYPE(dtype, ...)                                   \
     do {                                                                \

@@ -33,11 +33,11 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
     const T* __restrict__ q_norm_w, const T* __restrict__ k_norm_w, float eps, const float* __restrict__ cos_sin, int rotary,
     T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* positions, const int* slot_map,
     const int* cu_seqlens, const int* seq_slots, const int* kv_lens, int B, int nq, int nkv, int D, int V, int Dp, int page_size,
-    int write_kv, int head_norm) {
+    int write_kv, int head_norm, int shared_kv) {
     extern __shared__ float y[];                       // [channels]
     __shared__ float scratch[33];
     const int t = blockIdx.x;
-    const int Cq = nq * D, Ck = write_kv ? nkv * D : 0, Cv = write_kv ? nkv * V : 0, C = Cq + Ck + Cv;
+    const int Cq = nq * D, Ck = write_kv ? nkv * D : 0, Cv = write_kv && !shared_kv ? nkv * V : 0, C = Cq + Ck + Cv;
     const int p = __ldcg(positions + t);
     const int b = sequence_of(cu_seqlens, B, t);
     const int n_new = __ldcg(cu_seqlens + b + 1) - __ldcg(cu_seqlens + b);
@@ -82,6 +82,17 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         if (c < Cq) ssq = fmaf(acc, acc, ssq);
         else if (c < Cq + Ck) ssk = fmaf(acc, acc, ssk);
     }
+    const int sm = write_kv ? __ldcg(slot_map + t) : 0;
+    const int page = sm / page_size, off = sm - page * page_size;
+    if (write_kv && shared_kv) {
+        // The values are the keys' rows as they are here, before norm and rotation.
+        __syncthreads();
+        for (int e = threadIdx.x; e < nkv * Dp; e += CI_THREADS) {
+            const int head = e / Dp, d = e % Dp;
+            v_cache[(((size_t)page * nkv + head) * page_size + off) * Dp + d] = from_f32<T>(d < V ? y[Cq + head * D + d] : 0.f);
+        }
+        __syncthreads();
+    }
     if (head_norm) {
         // A warp per head: the order of a head's sum depends on the head's size alone.
         __syncthreads();
@@ -109,8 +120,6 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
     __syncthreads();
     const int half = rotary >> 1;
     const float* cs = cos_sin != nullptr ? cos_sin + (size_t)p * rotary : nullptr;       // [half][2] = (cos, sin)
-    const int sm = write_kv ? __ldcg(slot_map + t) : 0;
-    const int page = sm / page_size, off = sm - page * page_size;
     // Queries and keys: heads of Dp elements, the first D from y (rotated where the rotation reaches), zeros after.
     const int qk_heads = nq + (write_kv ? nkv : 0);
     for (int e = threadIdx.x; e < qk_heads * Dp; e += CI_THREADS) {
@@ -128,7 +137,7 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         if (head < nq) q_out[((size_t)t * nq + head) * Dp + d] = from_f32<T>(v);
         else k_cache[(((size_t)page * nkv + head - nq) * page_size + off) * Dp + d] = from_f32<T>(v);
     }
-    if (write_kv)
+    if (write_kv && !shared_kv)
         for (int e = threadIdx.x; e < nkv * Dp; e += CI_THREADS) {
             const int head = e / Dp, d = e % Dp;
             v_cache[(((size_t)page * nkv + head) * page_size + off) * Dp + d] = from_f32<T>(d < V ? y[Cq + Ck + head * V + d] : 0.f);
@@ -138,17 +147,19 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
 // proj [n, ld] of T: the step's projected rows, queries (nq * D) then, with write_kv, keys (nkv * D) and values (nkv * V);
 // bias and conv [channels, taps] in the same channel order (null: none; taps 0: no convolution); state [slots, taps - 1, channels]
 // float; cos_sin [positions, rotary / 2, 2] float (null: no rotation; pairs i, i + rotary / 2). head_norm: the norm weights are
-// [D] and every head is normed by itself.
+// [D] and every head is normed by itself. shared_kv: there are no value rows; a token's values are its keys' rows before norm and
+// rotation.
 extern "C" int ti_conv_attention_inputs(const void* proj, long long ld, const void* bias, const void* conv, int taps, const float* state,
                                         const void* q_norm_w, const void* k_norm_w, float eps, const float* cos_sin, int rotary, void* q_out,
                                         void* k_cache, void* v_cache, const int* positions, const int* slot_map, const int* cu_seqlens,
                                         const int* seq_slots, const int* kv_lens, int n, int B, int nq, int nkv, int D, int V, int Dp,
-                                        int page_size, int write_kv, int head_norm, int dtype, cudaStream_t stream) {
+                                        int page_size, int write_kv, int head_norm, int shared_kv, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
     TI_REQUIRE(taps >= 0 && taps <= CI_MAX_TAPS && (taps <= 1 || state != nullptr) && (taps == 0 || conv != nullptr), "conv_attention_inputs: %d taps", taps);
     TI_REQUIRE(D > 0 && V > 0 && Dp >= D && Dp >= V && nq > 0 && nkv > 0, "conv_attention_inputs: heads of %d / %d in rows of %d", D, V, Dp);
     TI_REQUIRE(cos_sin == nullptr || (rotary >= 2 && rotary % 2 == 0 && rotary <= D), "conv_attention_inputs: rotation over %d of %d", rotary, D);
-    const int C = nq * D + (write_kv ? nkv * (D + V) : 0);
+    TI_REQUIRE(!shared_kv || V == D, "conv_attention_inputs: values that are the keys' projection have the keys' size (%d, not %d)", D, V);
+    const int C = nq * D + (write_kv ? nkv * (shared_kv ? D : D + V) : 0);
     const size_t smem = (size_t)C * sizeof(float);
     TI_REQUIRE(smem <= 160 * 1024, "conv_attention_inputs: %d channels", C);
 #define CI_LAUNCH(TAPS)                                                                                                                       \
@@ -156,7 +167,7 @@ extern "C" int ti_conv_attention_inputs(const void* proj, long long ld, const vo
         if (smem > 48 * 1024) cudaFuncSetAttribute(conv_attention_inputs_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         ti_launch(conv_attention_inputs_kernel<T, TAPS>, dim3(n), dim3(CI_THREADS), smem, stream, (const T*)proj, ld, (const T*)bias, (const T*)conv,  \
                   taps, state, (const T*)q_norm_w, (const T*)k_norm_w, eps, cos_sin, rotary, (T*)q_out, (T*)k_cache, (T*)v_cache, positions,       \
-                  slot_map, cu_seqlens, seq_slots, kv_lens, B, nq, nkv, D, V, Dp, page_size, write_kv, head_norm);                               \
+                  slot_map, cu_seqlens, seq_slots, kv_lens, B, nq, nkv, D, V, Dp, page_size, write_kv, head_norm, shared_kv);                          \
     } while (0)
     TI_DISPATCH_DTYPE(dtype, {
         switch (taps) {

@@ -13,7 +13,8 @@ template <int D>
 __device__ __forceinline__ void decode_tile(const bf16* kt, const bf16* vt, const unsigned (&qf)[D / 16][4], float (&o)[D / 8][4],
                                             float& m0, float& m1, float& l0, float& l1, int tile, int warp, int lane,
                                             int kv_len, int first_key, float scale_log2e, const float* __restrict__ bias0 = nullptr,
-                                            const float* __restrict__ bias1 = nullptr, int bias_len = 0) {
+                                            const float* __restrict__ bias1 = nullptr, int bias_len = 0, const AttnExtras& ex = AttnExtras{},
+                                            float slope0 = 0.f, float slope1 = 0.f) {
     constexpr int CPR = D / 8, KS = D / 16, NT = D / 8;
     const int t = lane & 3;
         float s[2][4];
@@ -45,8 +46,17 @@ __device__ __forceinline__ void decode_tile(const bf16* kt, const bf16* vt, cons
                 const int dist = min(kv_len - 1 - key, bias_len - 1);
                 add0 = bias0[dist]; add1 = bias1[dist];
             }
-            s[nt][j] = ok ? fmaf(s[nt][j], scale_log2e, add0) : -INFINITY;
-            s[nt][2 + j] = ok ? fmaf(s[nt][2 + j], scale_log2e, add1) : -INFINITY;
+            if (ex.slope != nullptr) {
+                const float back = (float)(key - (kv_len - 1));
+                add0 = fmaf(slope0, back, add0); add1 = fmaf(slope1, back, add1);
+            }
+            if (ex.cap_out > 0.f) {
+                s[nt][j] = ok ? capped_score2(s[nt][j], ex) + add0 : -INFINITY;
+                s[nt][2 + j] = ok ? capped_score2(s[nt][2 + j], ex) + add1 : -INFINITY;
+            } else {
+                s[nt][j] = ok ? fmaf(s[nt][j], scale_log2e, add0) : -INFINITY;
+                s[nt][2 + j] = ok ? fmaf(s[nt][2 + j], scale_log2e, add1) : -INFINITY;
+            }
             mx0 = fmaxf(mx0, s[nt][j]);
             mx1 = fmaxf(mx1, s[nt][2 + j]);
         }

@@ -577,11 +577,22 @@ extern "C" int ti_history_update(float* hist, long long hist_stride, const void*
 }
 
 // ------------------------------------------------------------------------------------------------ a scan's output
-// y [n][H * V] of T = o / rms(o over a head) * w * silu(gate): every head normed by itself in 32-bit; w is [V] (one weight for all
-// heads, `shared_w`) or [H * V]; gate [n][ldg] of T holds the gate's projection. A warp per (token, head).
+// y [n][H * V] of T = o / rms(o over a head) * w * act(gate): every head normed by itself in 32-bit; w is [V] (one weight for all
+// heads, `shared_w`) or [H * V], or null (no weight); gate [n][ldg] of T holds the gate's projection, act is SiLU or, with
+// `gate_sigmoid`, the sigmoid. With nq and em [n][H] (a gated matrix memory) o is divided by max(|nq|, em) + 1e-6 first. With m_new [n][H]
+// (one-token steps) the sequences' running maxima at m_state + slot * state_stride are moved on. A warp per (token, head).
+struct HeadsOut {
+    const float* nq;
+    const float* em;
+    const float* m_new;
+    float* m_state;
+    long long state_stride;
+    const int* seq_slots;
+    int gate_sigmoid;
+};
 template <typename T>
 __global__ void heads_norm_gate_kernel(T* __restrict__ y, const float* o, const T* gate, long long ldg, const T* __restrict__ w, int shared_w,
-                                       float eps, int H, int V, size_t heads_total) {
+                                       float eps, int H, int V, size_t heads_total, HeadsOut ex) {
     pdl_enter();
     const int lane = threadIdx.x & 31;
     const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -589,25 +600,34 @@ __global__ void heads_norm_gate_kernel(T* __restrict__ y, const float* o, const 
     const size_t t = item / H;
     const int h = (int)(item % H);
     const float* src = o + (t * H + h) * V;
+    const float div = ex.nq != nullptr ? fmaxf(fabsf(__ldcg(ex.nq + item)), __ldcg(ex.em + item)) + 1e-6f : 1.f;
+    if (ex.m_new != nullptr && lane == 0) ex.m_state[(size_t)__ldcg(ex.seq_slots + t) * ex.state_stride + h] = __ldcg(ex.m_new + item);
     float ss = 0.f;
     for (int d = lane; d < V; d += 32) {
-        const float v = __ldcg(src + d);
+        const float v = __ldcg(src + d) / div;
         ss = fmaf(v, v, ss);
     }
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
     for (int d = lane; d < V; d += 32) {
-        float v = __ldcg(src + d) * inv * to_f32(w[shared_w ? d : h * V + d]);
-        if (gate != nullptr) v *= rs_silu(to_f32(__ldcg(gate + t * ldg + h * V + d)));
+        float v = __ldcg(src + d) / div * inv;
+        if (w != nullptr) v *= to_f32(w[shared_w ? d : h * V + d]);
+        if (gate != nullptr) {
+            const float g = to_f32(__ldcg(gate + t * ldg + h * V + d));
+            v *= ex.gate_sigmoid ? 1.0f / (1.0f + expf(-g)) : rs_silu(g);
+        }
         y[(t * H + h) * V + d] = from_f32<T>(v);
     }
 }
 
-extern "C" int ti_heads_norm_gate(void* y, const float* o, const void* gate, long long ldg, const void* w, int shared_w, float eps, int n, int H,
-                                  int V, int dtype, cudaStream_t stream) {
+extern "C" int ti_heads_norm_gate(void* y, const float* o, const void* gate, long long ldg, const void* w, int shared_w, float eps, const float* nq,
+                                  const float* em, const float* m_new, float* m_state, long long state_stride, const int* seq_slots,
+                                  int gate_sigmoid, int n, int H, int V, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
+    TI_REQUIRE((nq != nullptr) == (em != nullptr) && (m_new == nullptr || (m_state != nullptr && seq_slots != nullptr)), "heads_norm_gate: nq comes with em, m_new with a state");
+    const HeadsOut ex = {nq, em, m_new, m_state, state_stride, seq_slots, gate_sigmoid};
     const size_t total = (size_t)n * H;
     TI_DISPATCH_DTYPE(dtype, (ti_launch(heads_norm_gate_kernel<T>, dim3((unsigned)((total + 3) / 4)), dim3(128), 0, stream, (T*)y, o, (const T*)gate,
-                                        ldg, (const T*)w, shared_w, eps, H, V, total)));
+                                        ldg, (const T*)w, shared_w, eps, H, V, total, ex)));
     return ti_check_launch("heads_norm_gate");
 }
 

@@ -88,7 +88,8 @@ extern "C" int ti_router_topk(const void* h, const void* wr, const float* logits
 // A router with more rules. z [n, ldz] holds the 32-bit logits of `total` = experts + pass choices (and, with a gate, one more
 // column: the gate's logit); without z the kernel computes them from h and wr (rows in that order). Per token:
 //   s = softmax(z[0 .. total)) (or sigmoid of each), c = s + correction (the CHOICE score; correction may be null);
-//   the choices form `groups` equal groups of neighbours, a group's score is its largest c, only the `keep` best groups stay
+//   the choices form `groups` equal groups of neighbours, a group's score is its largest c (group_best 1) or the sum of its two
+//   largest (group_best 2), only the `keep` best groups stay
 //   (ties to the smaller index); of those the `top` largest c are chosen (ties to the smaller index);
 //   weight = s of the chosen, divided by (their sum + 1e-20) with `renormalize`.
 // ids [n, top + always]: the chosen expert, or -1 for a pass choice (the last `total - experts`: their output is the input
@@ -96,7 +97,7 @@ extern "C" int ti_router_topk(const void* h, const void* wr, const float* logits
 // sigmoid(gate logit), or 1 without a gate.
 template <typename T>
 __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const float* z_in, long long ldz, int width, int experts, int total,
-                                     int softmax, const float* __restrict__ correction, int groups, int keep, int top, int renormalize,
+                                     int softmax, const float* __restrict__ correction, int groups, int keep, int group_best, int top, int renormalize,
                                      int always, int gate, int* __restrict__ ids, float* __restrict__ scores, float* __restrict__ pass_weight) {
     __shared__ float z[RT_MAX_EXPERTS + 1], c[RT_MAX_EXPERTS], gs[RT_MAX_EXPERTS];
     __shared__ float scratch[33];
@@ -133,9 +134,12 @@ __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const
     const int per = total / groups;
     if (keep < groups) {
         for (int g = threadIdx.x; g < groups; g += RT_THREADS) {
-            float best = -INFINITY;
-            for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, c[e]);
-            gs[g] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                if (c[e] > best) { second = best; best = c[e]; }
+                else second = fmaxf(second, c[e]);
+            }
+            gs[g] = group_best >= 2 && per >= 2 ? best + second : best;
         }
         __syncthreads();
         // A group stays if fewer than `keep` groups come before it (a larger score, or an equal one with a smaller index).
@@ -189,16 +193,17 @@ __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const
 }
 
 extern "C" int ti_router_select(const void* h, const void* wr, const float* z, long long ldz, int n, int width, int experts, int total, int softmax,
-                                const float* correction, int groups, int keep, int top, int renormalize, int always, int gate, int* ids,
+                                const float* correction, int groups, int keep, int group_best, int top, int renormalize, int always, int gate, int* ids,
                                 float* scores, float* pass_weight, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
     TI_REQUIRE(experts >= 0 && total >= experts && total >= 1 && total <= RT_MAX_EXPERTS && top >= 1 && top <= total && always >= 0,
                "router_select: top %d of %d choices (%d experts)", top, total, experts);
     TI_REQUIRE(groups >= 1 && total % groups == 0 && keep >= 1 && keep <= groups && keep * (total / groups) >= top,
                "router_select: %d of %d groups over %d choices for top %d", keep, groups, total, top);
+    TI_REQUIRE(group_best == 1 || group_best == 2, "router_select: a group's score from its %d best", group_best);
     TI_REQUIRE(total == experts || pass_weight != nullptr, "router_select: pass choices need their weights' output");
     TI_DISPATCH_DTYPE(dtype, (ti_launch(router_select_kernel<T>, dim3(n), dim3(RT_THREADS), 0, stream, (const T*)h, (const T*)wr, z, ldz, width, experts,
-                                        total, softmax, correction, groups, keep, top, renormalize, always, gate, ids, scores, pass_weight)));
+                                        total, softmax, correction, groups, keep, group_best, top, renormalize, always, gate, ids, scores, pass_weight)));
     return ti_check_launch("router_select");
 }
 

@@ -91,6 +91,17 @@ class DecoderModel:
             if any(not 0 <= occ < len(spec.order) for occ in spec.pass_input.at):
                 raise ValueError(f"pass input before layer runs {spec.pass_input.at} of {len(spec.order)}")
         self._pass_starts = frozenset(spec.pass_input.at) if spec.pass_input is not None else frozenset()
+        # Arrangements that keep something per sequence themselves have cache entries after the embedding's, one per layer run.
+        self._block_requests, self._block_cache = [], {}
+        first = len(spec.order) + (self._embedding_request is not None)
+        for occ, li in enumerate(spec.order):
+            ask = getattr(self.blocks[li], "cache_request", None)
+            request = ask() if ask is not None else None
+            if request is not None:
+                self._block_cache[occ] = first + len(self._block_requests)
+                self._block_requests.append(request)
+        if self._block_cache and self.pass_input is not None:
+            raise ValueError("an arrangement with a state of its own does not read a stream that is rewritten between passes")
         # Called with (index of the layer run, the 32-bit or 16-bit stream after it) when set: for tests and debugging.
         self.observer = None
         self.status = torch.zeros(1, dtype=torch.int32, device=rt.device)
@@ -109,11 +120,19 @@ class DecoderModel:
 
     # ---- what the cache has to hold, one entry per position of ``order``
     def cache_requests(self):
-        """One entry per layer run; then one for the embedding, if it keeps something per sequence."""
+        """One entry per layer run; then one for the embedding and one per run of a block that keeps something per sequence."""
         out = [self.blocks[li].mixer.cache_request() for li in self.spec.order]
         if self._embedding_request is not None:
             out.append(self._embedding_request)
-        return out
+        return out + self._block_requests
+
+    def _input_norm(self, occ, step, cache):
+        """What makes the input of layer run ``occ`` out of the stream (where the run's block keeps something per sequence there: with it)."""
+        norm = self.blocks[self.spec.order[occ]].input_norm
+        bind = getattr(norm, "bind", None)
+        if bind is None:
+            return norm
+        return bind(cache.layer(self._block_cache[occ]) if occ in self._block_cache else None, step)
 
     def cache_shares(self) -> Dict[int, int]:
         """occurrence -> the earlier occurrence whose storage it reads."""
@@ -154,7 +173,8 @@ class DecoderModel:
 
         for b in self.blocks:
             visit([b.mixer, b.feed_forward, b.mixer_norm, b.feed_forward_norm, getattr(b, "token_input", None),
-                   getattr(b, "mixer_post_norm", None), getattr(b, "feed_forward_post_norm", None)])
+                   getattr(b, "mixer_post_norm", None), getattr(b, "feed_forward_post_norm", None), getattr(b, "gates", None),
+                   getattr(b, "gate_biases", None), getattr(b, "conv", None)])
         visit([self.final_norm, self.head, self.pass_input])
         return total
 
@@ -184,13 +204,13 @@ class DecoderModel:
             ops.streams_begin(stream, x, self.streams)
             x = stream
         order = spec.order
-        self.blocks[order[0]].input_norm.forward(x, h) if order else self.final_norm.forward(x, h)
+        (self._input_norm(0, step, cache) if order else self.final_norm).forward(x, h)
         for occ, li in enumerate(order):
             if occ in self._pass_starts:
                 # The stream is rewritten before this run; the normed input that the run before left is made again.
                 self.pass_input.forward(x)
                 self.blocks[li].input_norm.forward(x, h)
-            nxt = self.blocks[order[occ + 1]].input_norm if occ + 1 < len(order) else self.final_norm
+            nxt = self._input_norm(occ + 1, step, cache) if occ + 1 < len(order) else self.final_norm
             self.blocks[li].forward(x, h, step, cache.layer(occ), nxt, h)
             if self.observer is not None:
                 self.observer(occ, x)

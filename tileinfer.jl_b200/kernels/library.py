@@ -80,6 +80,7 @@ _SIGNATURES = {
     "ti_attention_inputs": [_P, _L, _P, _I, _L, _P, _P, _P, _P, _P, _F, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "ti_attention_plain": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "ti_attention_plain_biased": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P],
+    "ti_attention_plain_ruled": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _F, _P, _I, _P],
     "ti_gemm_plain": [_P, _L, _P, _L, _P, _I, _I, _I, _I, _F, _F, _F, _F, _I, _P],
     "ti_argmax": [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P],
     "ti_sample": [_P, _L, _I, _I, _F, _I, _F, _P, _P, _P, _P, _P],
@@ -163,6 +164,9 @@ _SIGNATURES_FAST["ti_attention_decode_sink"] = _SIGNATURES_FAST["ti_attention_de
 _SIGNATURES_FAST["ti_attention_prefill_biased"] = _SIGNATURES_FAST["ti_attention_prefill"][:-1] + [_P, _I, _P, _I, _P]
 _SIGNATURES_FAST["ti_attention_prefill_tc_biased"] = _SIGNATURES_FAST["ti_attention_prefill_tc"][:-1] + [_P, _I, _P, _I, _P]
 _SIGNATURES_FAST["ti_attention_decode_biased"] = _SIGNATURES_FAST["ti_attention_decode_shared"][:-1] + [_P, _I, _P, _I, _P]
+# ... and with a cap of the scores and a slope per head after those
+for _name in ("prefill", "prefill_tc", "decode"):
+    _SIGNATURES_FAST[f"ti_attention_{_name}_ruled"] = _SIGNATURES_FAST[f"ti_attention_{_name}_biased"][:-1] + [_F, _P, _P]
 _SIGNATURES_FAST["ti_attention_prefill_tc_sink"] = _SIGNATURES_FAST["ti_attention_prefill_tc"][:-1] + [_P, _P]
 _SIGNATURES.update(_SIGNATURES_FAST)
 
@@ -192,11 +196,11 @@ _SIGNATURES.update({
     "ti_lightning_scan": [_P, _P, _L, _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "ti_lightning_out": [_P, _P, _P, _L, _P, _F, _I, _I, _I, _P],
     "ti_conv_attention_inputs": [_P, _L, _P, _P, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I,
-                                 _I, _I, _P],
+                                 _I, _I, _I, _P],
     "ti_conv_state_update": [_P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _P],
     "ti_sigmoid_gate": [_P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P],
     "ti_sum_add_norm32": [_P, _P, _P, _I, _L, _P, _P, _I, _L, _P, _P, _I, _F, _I, _I, _I, _P],
-    "ti_router_select": [_P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P],
+    "ti_router_select": [_P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P],
     "ti_gated_act": [_P, _P, _I, _I, _I, _I, _P],
 })
 
@@ -219,6 +223,17 @@ _SIGNATURES.update({
     "ti_shift_blend": [_P, _P, _P, _I, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "ti_delta_inputs": [_P, _P, _L, _P, _I, _P, _L, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "ti_history_update": [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _P],
-    "ti_heads_norm_gate": [_P, _P, _P, _L, _P, _I, _F, _I, _I, _I, _I, _P],
+    "ti_heads_norm_gate": [_P, _P, _P, _L, _P, _I, _F, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _P],
     "ti_pair_combine": [_P, _P, _P, _I, _L, _P, _P, _I, _L, _P, _P, _I, _F, _F, _F, _I, _I, _I, _P],
+})
+
+# Gated additions to a stream normed in groups, a convolution over a step's rows; retention and the gated matrix memory.
+_SIGNATURES.update({
+    "ti_gated_add_norm32": [_P, _P, _P, _I, _L, _P, _P, _I, _P, _P, _P, _I, _L, _P, _P, _P, _F, _I, _P, _I, _P, _L, _P, _P, _I, _I, _I, _P],
+    "ti_conv_rows": [_P, _P, _P, _I, _P, _L, _P, _P, _I, _I, _I, _I, _P],
+    "ti_retention_scan": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _I, _P, _F, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ti_memory_gates": [_P, _P, _P, _L, _P, _F, _P, _L, _P, _P, _I, _I, _P],
+    "ti_memory_scan": [_P, _P, _P, _L, _I, _I, _I, _P, _L, _P, _F, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ti_memory_token": [_P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P, _L, _P, _P, _L, _P, _F, _P, _I, _P, _F, _F, _P, _I, _F, _P, _I, _I, _I, _I,
+                        _I, _P],
 })

@@ -133,12 +133,27 @@ def attention_inputs(qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, eps, rota
 
 
 def attention_plain(out, q, k_cache, v_cache, block_table, tok_slot, positions, scale, nq, nkv, head_dim,
-                    page_size, window=0, sink=None, chunk=0, distance_bias=None):
+                    page_size, window=0, sink=None, chunk=0, distance_bias=None, cap=0.0, slopes=None):
     """``sink`` [nq] float32: one more term exp(sink[head]) in every softmax's denominator (no key, no value). ``chunk`` > 0: a
     key is visible only inside the query's chunk of so many positions (counted from the sequence's start). ``distance_bias``
-    [nq, L] float32: entry [head, min(distance, L - 1)] is added to the scaled score."""
+    [nq, L] float32: entry [head, min(distance, L - 1)] is added to the scaled score. ``cap`` > 0: the scaled score s becomes
+    cap tanh(s / cap) before that; ``slopes`` [nq] float32: slopes[head] * distance is taken off."""
     if sink is not None:
         _need(sink, "sink", torch.float32)
+    if cap or slopes is not None:
+        for t, name in ((slopes, "slopes"), (distance_bias, "distance_bias")):
+            if t is not None:
+                _need(t, name, torch.float32)
+                if t.shape[0] != nq:
+                    raise KernelError(f"attention: {name} {tuple(t.shape)} for {nq} heads")
+        _need(out, "out"); _need(q, "q", out.dtype); _need(k_cache, "k_cache", out.dtype); _need(v_cache, "v_cache", out.dtype)
+        _need(block_table, "block_table", torch.int32); _need(tok_slot, "tok_slot", torch.int32); _need(positions, "positions", torch.int32)
+        check(lib().ti_attention_plain_ruled(out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(),
+                                             block_table.stride(0), tok_slot.data_ptr(), positions.data_ptr(), scale, q.shape[0], nq, nkv,
+                                             head_dim, page_size, window or 0, _ptr(sink), int(chunk or 0), _ptr(distance_bias),
+                                             distance_bias.shape[1] if distance_bias is not None else 0, cap, _ptr(slopes), dtype_code(out.dtype),
+                                             _stream()), "attention_plain")
+        return
     if chunk or distance_bias is not None:
         if distance_bias is not None:
             _need(distance_bias, "distance_bias", torch.float32)
@@ -513,10 +528,10 @@ def lightning_out(y, o, gate, w, eps):
 
 
 def conv_attention_inputs(rows, bias, conv, taps, state, q_norm_w, k_norm_w, eps, rotation, q_out, k_cache, v_cache, step, slot_map,
-                          nq, nkv, dim, vdim, padded, page_size, write_kv=True, head_norm=False):
+                          nq, nkv, dim, vdim, padded, page_size, write_kv=True, head_norm=False, shared_kv=False):
     """The step's projected rows (queries, then keys and values with ``write_kv``) -> bias, causal convolution over time (history
     from ``state`` [slots, taps - 1, channels] float32), whole-row RMS norms of q and k (``head_norm``: every head by itself, with
-    one weight of the head's size), rotation -> q_out [n, nq, padded] and the keys and values at ``slot_map`` in the pools. ``step``
+    one weight of the head's size), rotation (``shared_kv``: no value rows, the values are the keys' rows before norm and rotation) -> q_out [n, nq, padded] and the keys and values at ``slot_map`` in the pools. ``step``
     gives positions, cu_seqlens, seq_slots, kv_lens."""
     _need(rows, "rows", q_out.dtype, contiguous=False); _need(q_out, "q_out")
     cos_sin = rotation.cos_sin if rotation is not None else None
@@ -529,7 +544,7 @@ def conv_attention_inputs(rows, bias, conv, taps, state, q_norm_w, k_norm_w, eps
                                          eps, _ptr(cos_sin), rotary, q_out.data_ptr(), _ptr(k_cache), _ptr(v_cache), step.positions.data_ptr(),
                                          _ptr(slot_map), step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), step.kv_lens.data_ptr(),
                                          rows.shape[0], step.n_seqs, nq, nkv, dim, vdim, padded, page_size, int(bool(write_kv)),
-                                         int(bool(head_norm)), dtype_code(q_out.dtype), _stream()), "conv_attention_inputs")
+                                         int(bool(head_norm)), int(bool(shared_kv)), dtype_code(q_out.dtype), _stream()), "conv_attention_inputs")
 
 
 def conv_state_update(state, rows, bias, taps, step, channels):
@@ -550,9 +565,10 @@ def sigmoid_gate(y, attn, gate, heads, vdim, padded, per_head=False):
 
 
 def router_select(h, wr, logits, experts, total, top, ids, scores, pass_weight=None, softmax=True, correction=None, groups=1, keep=1,
-                  renormalize=True, always=0, gate=False):
+                  group_best=1, renormalize=True, always=0, gate=False):
     """The router with groups, a correction for the choice, normalised weights, pass-through choices and a gated always-on unit
-    (``csrc/routed_experts.cu``: router_select). ``logits`` [n, >= total (+ 1 with gate)] float32 or None (then from h and wr)."""
+    (``csrc/routed_experts.cu``: router_select). ``group_best`` 1 or 2: a group's score is its best choice score or the sum of its two
+    best. ``logits`` [n, >= total (+ 1 with gate)] float32 or None (then from h and wr)."""
     _need(h, "h"); _need(wr, "wr", h.dtype); _need(ids, "ids", torch.int32); _need(scores, "scores", torch.float32)
     n, width = h.shape
     if tuple(ids.shape) != (n, top + always) or ids.shape != scores.shape or wr.shape[0] != total + int(bool(gate)):
@@ -564,7 +580,7 @@ def router_select(h, wr, logits, experts, total, top, ids, scores, pass_weight=N
     if pass_weight is not None:
         _need(pass_weight, "pass_weight", torch.float32)
     check(lib().ti_router_select(h.data_ptr(), wr.data_ptr(), _ptr(logits), logits.stride(0) if logits is not None else 0, n, width, experts, total,
-                                 int(bool(softmax)), _ptr(correction), groups, keep, top, int(bool(renormalize)), always, int(bool(gate)),
+                                 int(bool(softmax)), _ptr(correction), groups, keep, group_best, top, int(bool(renormalize)), always, int(bool(gate)),
                                  ids.data_ptr(), scores.data_ptr(), _ptr(pass_weight), dtype_code(h.dtype), _stream()), "router_select")
 
 
@@ -682,16 +698,23 @@ def delta_scan(o, qkv, ba, a_log, dt_bias, state, step, heads, qk_heads, dim, vd
                               vdim, _stream()), "delta_scan")
 
 
-def heads_norm_gate(y, o, gate, w, eps, heads, vdim):
-    """y [n, heads * vdim] = o / rms(o over each head) * w * silu(gate); w [vdim] (shared by the heads) or [heads * vdim]."""
-    _need(y, "y"); _need(o, "o", torch.float32); _need(w, "w", y.dtype)
+def heads_norm_gate(y, o, gate, w, eps, heads, vdim, gate_sigmoid=False, divisor=None, moves=None):
+    """y [n, heads * vdim] = o / rms(o over each head) * w * act(gate); w [vdim] (shared by the heads), [heads * vdim] or None; act SiLU or,
+    with ``gate_sigmoid``, the sigmoid. ``divisor`` (nq, em), both [n, heads] float32: o is divided by max(|nq|, em) + 1e-6 first.
+    ``moves`` (m_new [n, heads] float32, m_state [slots, heads] strided view, seq_slots): a one-token step's running maxima are stored."""
+    _need(y, "y"); _need(o, "o", torch.float32)
     if gate is not None:
         _need(gate, "gate", y.dtype, contiguous=False)
-    if w.numel() not in (vdim, heads * vdim):
-        raise KernelError(f"heads_norm_gate: a weight of {w.numel()} for {heads} heads of {vdim}")
-    check(lib().ti_heads_norm_gate(y.data_ptr(), o.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0, w.data_ptr(),
-                                   int(w.numel() == vdim), eps, y.shape[0], heads, vdim, dtype_code(y.dtype),
-                                   _stream()), "heads_norm_gate")
+    if w is not None:
+        _need(w, "w", y.dtype)
+        if w.numel() not in (vdim, heads * vdim):
+            raise KernelError(f"heads_norm_gate: a weight of {w.numel()} for {heads} heads of {vdim}")
+    nq, em = divisor if divisor is not None else (None, None)
+    m_new, m_state, slots = moves if moves is not None else (None, None, None)
+    check(lib().ti_heads_norm_gate(y.data_ptr(), o.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(w),
+                                   int(w is not None and w.numel() == vdim and heads > 1), eps, _ptr(nq), _ptr(em), _ptr(m_new), _ptr(m_state),
+                                   m_state.stride(0) if m_state is not None else 0, _ptr(slots), int(bool(gate_sigmoid)), y.shape[0], heads, vdim,
+                                   dtype_code(y.dtype), _stream()), "heads_norm_gate")
 
 
 def pair_combine(out, a, b, wa, wb, eps, scale_a, scale_b, dtype):
@@ -701,3 +724,101 @@ def pair_combine(out, a, b, wa, wb, eps, scale_a, scale_b, dtype):
     n, size = out.shape
     check(lib().ti_pair_combine(out.data_ptr(), *_rows_or_partials(a, dtype, "a"), *_rows_or_partials(b, dtype, "b"), _ptr(wa), _ptr(wb),
                                 int(wa is not None), eps, scale_a, scale_b, n, size, dtype_code(dtype), _stream()), "pair_combine")
+
+
+# ---------------------------------------------------------------- a stream whose sublayers are added through a gate; matrix memories
+def _branch_args(d, dtype, name):
+    """(rows, partials, parts, stride) of [n, size] rows of ``dtype`` (the rows may be strided) or 32-bit partial sums [s, n, size]."""
+    if d is None:
+        return (None, None, 0, 0)
+    if d.dim() == 3:
+        _need(d, name, torch.float32)
+        return (None, d.data_ptr(), d.shape[0], d.stride(0))
+    _need(d, name, dtype, contiguous=False)
+    if d.stride(1) != 1:
+        raise KernelError(f"{name} must have dense rows")
+    return (d.data_ptr(), None, 0, d.stride(0))
+
+
+def gated_add_norm32(x, d, gate, h, w, eps, groups=1, d_bias=None, gate_bias=None, index=None, scores=None, conv=None):
+    """x += (d + d_bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``d`` None: x stays as it is; ``gate`` None: no gate), then
+    h = x normed by its root mean square in ``groups`` equal parts, times w. ``d``: rows [n, size], 32-bit partial sums [s, n, size], or
+    with ``index`` and ``scores`` [n, per_row] rows still apart, of which row t's are added up. ``conv`` (weights [taps, size], history view
+    [slots, >= (taps - 1) * size] float32 or None, seq_slots, out): one-token steps only, out = h + conv(h), the history moved on."""
+    _need(x, "x", torch.float32); _need(h, "h"); _need(w, "w", h.dtype)
+    n, size = x.shape
+    c = (None, 0, None, 0, None, None)
+    if conv is not None:
+        cw, hist, slots, out = conv
+        _need(cw, "conv", h.dtype); _need(out, "conv_out", h.dtype)
+        if cw.shape[0] > 1:
+            _need(hist, "history", torch.float32, contiguous=False); _need(slots, "seq_slots", torch.int32)
+        c = (cw.data_ptr(), cw.shape[0], _ptr(hist) if cw.shape[0] > 1 else None, hist.stride(0) if cw.shape[0] > 1 else 0, slots.data_ptr(), out.data_ptr())
+    if index is not None:
+        _need(index, "index", torch.int32); _need(scores, "scores", torch.float32)
+    check(lib().ti_gated_add_norm32(x.data_ptr(), *_branch_args(d, h.dtype, "d"), _ptr(index), _ptr(scores), index.shape[1] if index is not None else 0,
+                                    _ptr(d_bias), *_branch_args(gate, h.dtype, "gate"), _ptr(gate_bias), h.data_ptr(), w.data_ptr(), eps, groups, *c,
+                                    n, size, dtype_code(h.dtype), _stream()), "gated_add_norm32")
+
+
+def conv_rows(out, h, conv, hist, step):
+    """out = h + conv(h) over a step's rows, conv [taps, size] causal per channel, earlier rows from the sequences' history ``hist``
+    [slots, >= (taps - 1) * size] float32 (None with one tap); ``history_update`` moves the history on afterwards."""
+    _need(out, "out"); _need(h, "h", out.dtype); _need(conv, "conv", out.dtype)
+    if hist is not None:
+        _need(hist, "history", torch.float32, contiguous=False)
+    n, size = h.shape
+    check(lib().ti_conv_rows(out.data_ptr(), h.data_ptr(), conv.data_ptr(), conv.shape[0], _ptr(hist), hist.stride(0) if hist is not None else 0,
+                             step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), n, step.n_seqs, size, dtype_code(h.dtype), _stream()), "conv_rows")
+
+
+def _rotation_args(rotation, step):
+    if rotation is None:
+        return (None, 0, step.positions.data_ptr())
+    if rotation.interleaved:
+        raise KernelError("matrix memories: only the half-split pairing is built")
+    return (rotation.cos_sin.data_ptr(), int(rotation.rotary_dim), step.positions.data_ptr())
+
+
+def retention_scan(o, rows, q_off, k_off, v_off, state, decay, rotation, q_scale, k_scale, step, heads, dim, vdim):
+    """S = decay_h S + k v^T, o = S^T q over the step's tokens, q and k rotated by position and scaled; ``state`` [slots, >= heads * dim * vdim]
+    float32 (rows may be strided); o [n, heads * vdim] float32."""
+    _need(o, "o", torch.float32); _need(rows, "rows", contiguous=False); _need(state, "state", torch.float32, contiguous=False)
+    _need(decay, "decay", torch.float32)
+    check(lib().ti_retention_scan(o.data_ptr(), rows.data_ptr(), rows.stride(0), q_off, k_off, v_off, state.data_ptr(), state.stride(0), decay.data_ptr(),
+                                  *_rotation_args(rotation, step), q_scale, k_scale, step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(),
+                                  rows.shape[0], step.n_seqs, heads, dim, vdim, dtype_code(rows.dtype), _stream()), "retention_scan")
+
+
+def memory_gates(coef, em, z, bias, cap, state, m_off, step, heads):
+    """coef [n, heads, 2] = (keep, add) and em [n, heads] = exp(-m) of the gated cell from the gate logits z [n, 2 heads] float32 (i, then f)
+    and their biases; m lies at ``m_off`` in the rows of ``state`` and moves on."""
+    _need(coef, "coef", torch.float32); _need(em, "em", torch.float32); _need(z, "z", torch.float32, contiguous=False)
+    _need(bias, "bias", torch.float32); _need(state, "state", torch.float32, contiguous=False)
+    check(lib().ti_memory_gates(coef.data_ptr(), em.data_ptr(), z.data_ptr(), z.stride(0), bias.data_ptr(), cap, state.data_ptr() + 4 * m_off,
+                                state.stride(0), step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), step.n_seqs, heads, _stream()), "memory_gates")
+
+
+def memory_scan(o, nq, rows, q_off, k_off, v_off, state, coef, q_scale, k_scale, step, heads, dim, vdim):
+    """S = keep S + add k v^T, n = keep n + add k, o = S^T q (not yet divided), nq = n . q over the step's tokens."""
+    _need(o, "o", torch.float32); _need(nq, "nq", torch.float32); _need(rows, "rows", contiguous=False); _need(coef, "coef", torch.float32)
+    _need(state, "state", torch.float32, contiguous=False)
+    check(lib().ti_memory_scan(o.data_ptr(), nq.data_ptr(), rows.data_ptr(), rows.stride(0), q_off, k_off, v_off, state.data_ptr(), state.stride(0),
+                               coef.data_ptr(), q_scale, k_scale, step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), rows.shape[0], step.n_seqs,
+                               heads, dim, vdim, dtype_code(rows.dtype), _stream()), "memory_scan")
+
+
+def memory_token(rows, offs, state, step, heads, dim, vdim, y=None, o=None, outs=(None, None, None), decay=None, z=None, bias=None, cap=0.0,
+                 rotation=None, q_scale=1.0, k_scale=1.0, w=None, gate_sigmoid=False, eps=1e-6) -> bool:
+    """One token per sequence of retention (``decay``) or of the gated cell (``z``, ``bias``, ``cap``): ``y`` the normed and gated heads
+    (value sizes up to 128), or ``o`` the raw ones with ``outs`` = (nq, em, m_new). ``offs``: columns of q, k, v and the output gate.
+    False for sizes the kernel refuses."""
+    _need(rows, "rows", contiguous=False); _need(state, "state", torch.float32, contiguous=False)
+    rc = lib().ti_memory_token(_ptr(y), _ptr(o), *(_ptr(t) for t in outs), rows.data_ptr(), rows.stride(0), *offs, state.data_ptr(), state.stride(0),
+                               _ptr(decay), _ptr(z), z.stride(0) if z is not None else 0, _ptr(bias), cap, *_rotation_args(rotation, step), q_scale,
+                               k_scale, _ptr(w), int(bool(gate_sigmoid)), eps, step.seq_slots.data_ptr(), step.n_seqs, heads, dim, vdim,
+                               dtype_code(rows.dtype), _stream())
+    if rc == 2:
+        return False
+    check(rc, "memory_token")
+    return True

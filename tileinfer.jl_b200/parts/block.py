@@ -3,6 +3,7 @@ h = norm1(x), on a 32-bit stream.
 ``post_norm``: x += m norm1(mixer(x)); x += m norm2(ffn(x)); x += m token_input(x), on a 32-bit stream.
 ``sandwich``: x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))), on a 32-bit stream.
 ``hyper``: pre-norm sublayers that read, rewrite and write to several copies of a 32-bit stream through learned tables.
+``gated``: pre-norm sublayers added to a 32-bit stream through learned gates, with a short causal convolution ahead of the mixer.
 
 Each residual add is fused with the norm that follows it, so a block receives the already
 normed input ``h`` and produces the next block's normed input with ``next_norm`` (the next
@@ -15,7 +16,8 @@ import torch
 
 from ..config.spec import TensorDecl
 from ..kernels import ops
-from .base import register_block
+from .base import CacheRequest, Part, register_block
+from .linear import Linear
 from .norm import StreamCast
 
 
@@ -221,4 +223,101 @@ class HyperBlock:
         delta = self.feed_forward.forward(h, step)
         blend, (w, b, eps, centred) = self._next(next_norm)
         ops.streams_update(x, delta, M2, c2, blend, h_out, w, b, eps, centred)
+        return h_out
+
+
+class ConvolvedRead:
+    """Stands where a ``gated`` block's input norm would: h = norm(x) and, ahead of the mixer, hc = h + conv(h), conv a causal convolution
+    over time per channel (weights [taps, size], tap taps - 1 on the token itself). The earlier rows of a step's first tokens are a small
+    state of the sequence, which the decoder hands over for every layer run (``bind``). In one-token steps the kernel that updates the
+    stream does norm and convolution as well. hc is left in the scratch buffer ``OUT``, where the block's ``forward`` finds it."""
+
+    OUT = "block.convolved"
+
+    def __init__(self, norm, conv, rt, cache=None, step=None):
+        self.norm, self.conv, self.rt, self.cache, self.step = norm, conv, rt, cache, step
+
+    def bind(self, cache, step):
+        return ConvolvedRead(self.norm, self.conv, self.rt, cache, step)
+
+    def forward(self, x, out):
+        return self.gated_add(x, None, out)
+
+    def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None):
+        taps, size = self.conv.shape
+        hist = self.cache.state.view(self.cache.state.shape[0], -1) if taps > 1 else None
+        convolved = self.rt.buffer(self.OUT, tuple(out.shape))
+        if self.step.is_decode:
+            return self.norm.gated_add(x, delta, out, gate, bias, gate_bias, conv=(self.conv, hist, self.step.seq_slots, convolved))
+        self.norm.gated_add(x, delta, out, gate, bias, gate_bias)
+        ops.conv_rows(convolved, out, self.conv, hist, self.step)
+        if taps > 1:
+            ops.history_update(hist, out, taps, self.step, size)
+        return out
+
+
+@register_block("gated")
+class GatedBlock(Part):
+    """Pre-norm sublayers on a 32-bit stream, each multiplied by a gate before it is added (a layer may have no feed-forward):
+
+        h = norm1(x);   x += mixer(h + conv(h)) * sigmoid(R1 h + b1)
+        h = norm2(x);   x += ffn(h) * sigmoid(R2 h + b2)
+
+    The gates read h as the norm left it, before the convolution. Options: ``taps`` (0: no convolution, the mixer reads h) with ``conv``
+    the name of its weights [size, taps]; ``gates``: the names of R1 and R2 [size, size], whose biases have ``bias_suffix`` added (None:
+    no gates). A mixer whose output projection has a bias (``out_bias``) leaves it to the kernel that updates the stream; a
+    routed feed-forward leaves a token's rows apart for it. The norms are of a kind that offers ``gated_add`` (``rmsnorm32``)."""
+
+    def __init__(self, spec, mixer, feed_forward, mixer_norm, feed_forward_norm, tensors, rt):
+        self.spec, self.rt = spec, rt
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
+        o = spec.options
+        self.taps = int(o.get("taps") or 0)
+        # Kept [taps, size]: neighbouring channels' weights of one tap lie together.
+        self.conv = rt.param(tensors[o["conv"]]).t().contiguous() if self.taps else None
+        if hasattr(feed_forward, "rows_apart"):
+            feed_forward.rows_apart = True
+        self.gates, self.gate_biases = [], []
+        for name in (o.get("gates") or ())[:2 if feed_forward is not None else 1]:
+            gate = Linear(rt.param(tensors[name]), rt, "residual_gate")
+            gate.partials_name = "residual_gate.partials"
+            self.gates.append(gate)
+            self.gate_biases.append(rt.param(tensors[name + o["bias_suffix"]]))
+        self._read = ConvolvedRead(mixer_norm, self.conv, rt) if self.taps else mixer_norm
+
+    @classmethod
+    def tensors(cls, spec):
+        o, W = spec.options, spec.mixer.hidden_size
+        out = []
+        if int(o.get("taps") or 0):
+            out.append(TensorDecl(o["conv"], (W, int(o["taps"])), ("normal", 0.3)))
+        for name in (o.get("gates") or ())[:2 if spec.feed_forward is not None else 1]:
+            out += [TensorDecl(name, (W, W), ("normal", W ** -0.5)), TensorDecl(name + o["bias_suffix"], (W,), ("normal", 0.5))]
+        return out
+
+    def cache_request(self):
+        """The last taps - 1 rows that the convolution read, per layer run."""
+        return CacheRequest("state", shape=(self.taps - 1, self.spec.mixer.hidden_size), dtype=torch.float32) if self.taps > 1 else None
+
+    @property
+    def input_norm(self):
+        return self._read
+
+    def _gate(self, i, h):
+        if not self.gates:
+            return {}
+        z = self.gates[i].forward(h, self.rt.buffer("residual_gate.rows", tuple(h.shape)), allow_partials=True)
+        return {"gate": z, "gate_bias": self.gate_biases[i]}
+
+    def forward(self, x, h, step, cache, next_norm, h_out):
+        gate = self._gate(0, h)
+        delta = self.mixer.forward(self.rt.buffer(ConvolvedRead.OUT, tuple(h.shape)) if self.taps else h, step, cache)
+        bias = getattr(self.mixer, "out_bias", None)
+        if self.feed_forward is None:
+            next_norm.gated_add(x, delta, h_out, bias=bias, **gate)
+            return h_out
+        self.feed_forward_norm.gated_add(x, delta, h, bias=bias, **gate)
+        gate = self._gate(1, h)
+        next_norm.gated_add(x, self.feed_forward.forward(h, step), h_out, **gate)
         return h_out

@@ -30,9 +30,13 @@ logarithmic steps up to ``far``, the last row from there on. In bfloat16 attenti
 library's paged kernels (tensor-memory and ``mma.sync`` prompt kernels, split-KV decode kernel; the bias comes as a table by distance),
 in 32-bit in the plain kernel.
 
+``shared_kv``: there is no value projection; a token's values are its keys as projected (bias and convolution included), before norm and
+rotation. ``softcap`` c: the scaled score s becomes c tanh(s / c) before any bias. ``slopes`` (one number per head): slope * (i - j) is
+taken off the score after the cap, a linear bias by distance. Both run in every paged kernel.
+
 Record: ``num_heads``, ``num_kv_heads``, ``head_dim``, ``scale``, ``window``, ``kv_source``, ``qk_norm_eps`` and the options
 ``value_dim``, ``conv_taps`` (0: none), ``bias``, ``out_bias``, ``row_norm``, ``head_norm``, ``norm_weight``, ``sink``, ``gate``,
-``chunk``, ``distance_bias``.
+``chunk``, ``distance_bias``, ``shared_kv``, ``softcap``, ``slopes``.
 """
 from __future__ import annotations
 
@@ -80,10 +84,13 @@ class ConvAttention(Mixer):
             raise ValueError(f"conv_attention: heads of {self.dim} / {self.vdim} exceed the attention kernels' {ops.MAX_HEAD_DIM}")
         n, p = spec.tensor_names, spec.prefix
         get = lambda name: rt.param(tensors[p + name])
-        kinds = ["q", "k", "v"] if self.own_kv else ["q"]
+        self.shared_kv = bool(o.get("shared_kv", False))
+        if self.shared_kv and self.vdim != self.dim:
+            raise ValueError(f"conv_attention: values that are the keys have the keys' size {self.dim}, not {self.vdim}")
+        kinds = (["q", "k"] if self.shared_kv else ["q", "k", "v"]) if self.own_kv else ["q"]
         mats = [get(n[k]) for k in kinds] + ([get(n["g"])] if self.gated else [])
         self.proj = Linear(torch.cat(mats, 0).contiguous(), rt, "conv_attention_in")
-        self.channels = self.nq * self.dim + (self.nkv * (self.dim + self.vdim) if self.own_kv else 0)
+        self.channels = self.nq * self.dim + (self.nkv * (self.dim if self.shared_kv else self.dim + self.vdim) if self.own_kv else 0)
         self.bias = torch.cat([get(n[k] + n["bias_suffix"]) for k in kinds]).contiguous() if self.bias_on else None
         self.conv = torch.cat([get(n[k] + n["conv_suffix"]) for k in kinds], 0).contiguous() if self.taps else None
         self.head_norm = bool(o.get("head_norm", False))
@@ -109,6 +116,14 @@ class ConvAttention(Mixer):
             index = torch.tensor(distance_buckets(rel.shape[0], far, count), dtype=torch.long, device=rel.device)
             self.distance_bias = rel[index].t().contiguous()                          # [heads, count]: the bias by distance
             self.distance_bias2 = (self.distance_bias * 1.4426950408889634).contiguous()      # for the kernels that work in base 2
+        self.softcap = float(o.get("softcap") or 0.0)
+        self.slopes = self.slopes2 = None
+        if o.get("slopes"):
+            if len(o["slopes"]) != self.nq:
+                raise ValueError(f"conv_attention: {len(o['slopes'])} slopes for {self.nq} heads")
+            exact = torch.tensor([float(v) for v in o["slopes"]], dtype=torch.float64)
+            self.slopes = exact.float().to(rt.device)
+            self.slopes2 = (exact * 1.4426950408889634).float().to(rt.device)          # for the kernels that work in base 2
         self.out_name, self.gated_name = "mixer.delta", "conv_attention.gated"
         self.sink = rt.param(tensors[p + n["sink"]], keep_dtype=True).float().contiguous() if self.sink_on else None
         self.o = Linear(get(n["o"]), rt, "o")
@@ -126,7 +141,7 @@ class ConvAttention(Mixer):
         std = lambda fan_in: ("normal", fan_in ** -0.5)
         rows = {"q": H * D}
         if spec.kv_source is None:
-            rows.update({"k": G * D, "v": G * V})
+            rows.update({"k": G * D} if o.get("shared_kv", False) else {"k": G * D, "v": G * V})
         out = [TensorDecl(p + n["o"], (W, H * V), std(H * V))]
         if o.get("out_bias", False):
             out.append(TensorDecl(p + n["o"] + n["bias_suffix"], (W,), ("normal", 0.1)))
@@ -170,17 +185,19 @@ class ConvAttention(Mixer):
         meta = step.group(cache.group_index)
         ops.conv_attention_inputs(rows, self.bias, self.conv, self.taps, cache.state, self.q_norm, self.k_norm, s.qk_norm_eps, self.rotation,
                                   q, cache.k, cache.v, step, meta.slot_mapping, nq, nkv, D, V, Dp, cache.page_size, write_kv=self.own_kv,
-                                  head_norm=self.head_norm)
+                                  head_norm=self.head_norm, shared_kv=self.shared_kv)
         if self.taps > 1:
             ops.conv_state_update(cache.state, rows, self.bias, self.taps, step, C)
         attn = rt.buffer("attention.out", (n, nq * Dp))
         done = False
         if rt.fast:
             from ..kernels import fast
-            done = fast.attention(attn, q, cache, meta, step, self.attn_spec, sink=self.sink, chunk=self.chunk, distance_bias2=self.distance_bias2)
+            done = fast.attention(attn, q, cache, meta, step, self.attn_spec, sink=self.sink, chunk=self.chunk, distance_bias2=self.distance_bias2,
+                                  cap=self.softcap, slopes2=self.slopes2)
         if not done:
             ops.attention_plain(attn, q, cache.k, cache.v, meta.block_table, step.tok_slot, step.positions, s.scale, nq, nkv, Dp,
-                                cache.page_size, window=s.window or 0, sink=self.sink, chunk=self.chunk, distance_bias=self.distance_bias)
+                                cache.page_size, window=s.window or 0, sink=self.sink, chunk=self.chunk, distance_bias=self.distance_bias,
+                                cap=self.softcap, slopes=self.slopes)
         if self.gated or Dp != V:
             y = rt.buffer(self.gated_name, (n, nq * V))
             ops.sigmoid_gate(y, attn, rows[:, C:] if self.gated else None, nq, V, Dp, per_head=self.gate_per_head)

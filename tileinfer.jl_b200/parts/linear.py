@@ -30,3 +30,13 @@ class Linear:
                 return done
         ops.gemm_plain(out, x, self.weight, epilogue, act)
         return out
+
+    def forward_f32(self, x: torch.Tensor, out: torch.Tensor):
+        """Writes the 32-bit sums to ``out`` [n, out] float32, not rounded to the element type where a fast kernel takes the sizes."""
+        if self.rt.fast:
+            from ..kernels import fast
+            done = fast.linear_f32(self, x, out)
+            if done is not None:
+                return done
+        ops.gemm_plain(out, x, self.weight, ops.EPI_F32_OUT)
+        return out

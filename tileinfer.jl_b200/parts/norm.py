@@ -40,13 +40,19 @@ class RMSNorm32(Norm):
 
     Besides ``forward`` it serves blocks that normalise a sublayer's OUTPUT: ``branch_add(x, delta, mult, h, next_norm)``
     does x += mult * norm(delta) on a 32-bit stream and, in the same kernel, prepares the next reader's input
-    (``next_norm``: another norm of this kind or a :class:`StreamCast`)."""
+    (``next_norm``: another norm of this kind or a :class:`StreamCast`).
+
+    Option ``groups`` g: the row is split into g equal consecutive parts and each is divided by its own root mean square. It is built for
+    the blocks that add sublayers through ``gated_add``; the kernels of the other arrangements refuse such a norm."""
 
     def __init__(self, spec: NormSpec, tensors, rt):
         self.spec, self.rt = spec, rt
         self.weight = rt.param(tensors[spec.weight_name])
         self.eps = float(spec.eps)
         self.offset = bool(spec.options.get("offset", False))
+        self.groups = int(spec.options.get("groups") or 1)
+        if self.groups < 1 or spec.size % self.groups:
+            raise ValueError(f"{spec.weight_name}: {spec.size} elements do not divide into {self.groups} groups")
 
     @classmethod
     def tensors(cls, spec: NormSpec):
@@ -54,20 +60,41 @@ class RMSNorm32(Norm):
         init = ("normal", std) if spec.options.get("offset", False) else ("one_plus_normal", std)
         return [TensorDecl(spec.weight_name, (spec.size,), init)]
 
+    def _one_group(self, what):
+        if self.groups != 1:
+            raise NotImplementedError(f"a norm in {self.groups} groups does not serve {what}")
+
     def out_args(self):
+        self._one_group("as the next norm of branch_add")
         return (self.weight, self.eps, self.offset)
 
+    def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None, conv=None):
+        """x += (delta + bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``delta`` None: x stays), then out = norm(x). ``delta``:
+        rows, 32-bit partial sums or :class:`GatheredRows` with weights; ``gate``: rows or partial sums, None for no gate. ``conv``: see
+        ``ops.gated_add_norm32``."""
+        if self.offset:
+            raise NotImplementedError("a gain stored minus one, or a mean taken off, is not built for gated_add")
+        if isinstance(delta, GatheredRows):
+            ops.gated_add_norm32(x, delta.rows, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, delta.index, delta.scores, conv)
+        else:
+            ops.gated_add_norm32(x, delta, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, conv=conv)
+        return out
+
     def forward(self, x, out):
+        if self.groups != 1:
+            return self.gated_add(x, None, out)
         ops.norm32(out, x, self.weight, self.eps, self.offset)
         return out
 
     def sum_add(self, x, d1, d2, out):
         """x += d1 + d2 on a 32-bit stream (two sublayers that read the same input; ``d2`` may be None), then out = norm(x)."""
+        self._one_group("blocks that add two sublayers at once")
         ops.sum_add_norm32(x, d1, d2, out, self.weight, self.eps, self.offset)
         return out
 
     def branch_add(self, x, delta, mult, h=None, next_norm=None, bias=None):
         """``bias`` [size]: a vector added to ``delta`` before its norm (the bias of the product that made ``delta``)."""
+        self._one_group("on a sublayer's output")
         out_norm = next_norm.out_args() if next_norm is not None else None
         if isinstance(delta, GatheredRows):
             ops.branch_norm_add32(x, delta.rows, self.weight, self.eps, mult, self.offset, h, out_norm, gather=delta.index, bias=bias)
@@ -127,10 +154,11 @@ class LayerNorm32(RMSNorm32):
 
 class GatheredRows:
     """A sublayer's output that is still in pieces: row t is the sum of the rows ``index[t, :]`` of ``rows`` (the units a
-    token went through). A norm that offers ``branch_add`` adds them up while it reads them."""
+    token went through), with ``scores`` each times its weight. A norm that offers ``branch_add`` adds them up while it reads them,
+    one that offers ``gated_add`` does so with weights."""
 
-    def __init__(self, rows, index):
-        self.rows, self.index = rows, index
+    def __init__(self, rows, index, scores=None):
+        self.rows, self.index, self.scores = rows, index, scores
 
 
 class StreamCast(Norm):

@@ -16,11 +16,13 @@ Options of the record: ``experts``, ``top``, ``limit`` (None: no clamp), ``sigmo
     ``score`` "softmax": s = softmax(z) over all router outputs instead of sigmoid(z)
     ``correction``: a tensor added to s for the CHOICE only (the weights use s)
     ``groups`` (count, keep): the router's outputs form `count` equal groups of neighbours, a group's score is its largest choice
-        score, and only members of the `keep` best groups can be chosen
+        score, or with ``group_best`` 2 the sum of its two largest, and only members of the `keep` best groups can be chosen
     ``renormalize``: weights = the chosen s divided by (their sum + 1e-20)
     ``pass_through``: the last so many router outputs are not experts: a token that chooses one gets its own input back, times
         the weight (they take part in softmax, groups and the sum like any other)
-    ``shared_gate``: a tensor [1, width]; the shared unit's output is multiplied by sigmoid(shared_gate . h), one number per token Tensor names: ``router``, ``expert`` (a prefix pattern with ``{}`` for the expert's number), ``shared``
+    ``shared_gate``: a tensor [1, width]; the shared unit's output is multiplied by sigmoid(shared_gate . h), one number per token
+
+Tensor names: ``router``, ``expert`` (a prefix pattern with ``{}`` for the expert's number), ``shared``
 (a prefix), and inside a unit ``gate``, ``up``, ``down``.
 
 On the device the (token, choice) pairs are grouped by expert and every expert's rows go through its matrices in
@@ -60,6 +62,9 @@ class RoutedExperts(FeedForward):
         self.softmax, self.renormalize = o.get("score", "sigmoid") == "softmax", bool(o.get("renormalize", False))
         self.pass_through = int(o.get("pass_through", 0))
         self.groups, self.keep = (int(v) for v in (o.get("groups") or (1, 1)))
+        self.group_best = int(o.get("group_best", 1))
+        # Set by a block whose stream update adds up a token's rows itself: the output then comes as GatheredRows with their weights.
+        self.rows_apart = False
         if o.get("score", "sigmoid") not in ("sigmoid", "softmax"):
             raise ValueError(f"routed_experts: score {o.get('score')!r} (known: sigmoid, softmax)")
         if self.select and self.scale_input:
@@ -147,7 +152,7 @@ class RoutedExperts(FeedForward):
         if self.select:
             pass_weight = rt.buffer("experts.pass_weight", (n,), torch.float32) if self.pass_through else None
             ops.router_select(h, self.router, logits, E, E + self.pass_through, top, ids, scores, pass_weight, softmax=self.softmax,
-                              correction=self.correction, groups=self.groups, keep=self.keep, renormalize=self.renormalize,
+                              correction=self.correction, groups=self.groups, keep=self.keep, group_best=self.group_best, renormalize=self.renormalize,
                               always=self.always, gate=self.gate_on)
         else:
             ops.router_topk(h, self.router, top, ids, scores, logits, always=self.always)
@@ -168,6 +173,8 @@ class RoutedExperts(FeedForward):
             ops.grouped_gemm(ys, act, self.down, plan, tile)
         if self.scale_input:
             return GatheredRows(ys, pair_row)    # the norm that reads the output adds a token's rows up itself
+        if self.rows_apart and pass_weight is None:
+            return GatheredRows(ys, pair_row, scores)
         out = rt.buffer("feed_forward.delta", (n, W))
         ops.expert_combine(out, ys, pair_row, scores, None, per_token, scale_output=True, h=h if pass_weight is not None else None,
                            pass_weight=pass_weight)
