@@ -231,7 +231,7 @@ static int launch_lightning_scan(const char* what, float* o, const void* qkv, lo
         constexpr int VEC = 16 / (int)sizeof(T);                                                                                     \
         const bool vectors = aligned16(qkv) && ld % VEC == 0 && q_off % VEC == 0 && k_off % VEC == 0 && v_off % VEC == 0 &&          \
                              LS_TOKENS * (D / VEC) <= 4 * LS_COLS * PARTS;                                                           \
-        if (smem > 48 * 1024) {                                                                                                      \
+        if (smem > 40 * 1024) {                                                                                                      \
             cudaFuncSetAttribute(lightning_scan_kernel<T, DP, true, PARTS, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             cudaFuncSetAttribute(lightning_scan_kernel<T, DP, false, PARTS, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         }                                                                                                                            \
