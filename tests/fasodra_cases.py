@@ -188,7 +188,7 @@ class Recorder:
 
     def __init__(self, engine, cfg):
         self.engine = engine
-        self.tops = [l["mlp"]["router"]["top"] if l.get("mlp") else 0 for l in cfg["layers"]]
+        self.tops = [(l.get("mlp") or {}).get("router", {}).get("top", 0) for l in cfg["layers"]]
         self.rows, self.choices = [], {}
         engine.model.observer = self
 

@@ -94,7 +94,7 @@ def attention(h, w, p, m, eps):
 
 def retention(h, w, p, m, eps):
     t = h.shape[0]
-    H, D, V = m["heads"], m["dim"], m["vdim"]
+    H, D, V = m["heads"], m["dim"], m.get("vdim") or m["dim"]
     q, k = (h @ w[p + "q"].T).view(t, H, D), (h @ w[p + "k"].T).view(t, H, D)
     v = (h @ w[p + "v"].T).view(t, H, V)
     rot, pos = m.get("rot"), torch.arange(t)
@@ -130,7 +130,7 @@ def mlstm_cell(q, k, v, ig, fg):
 
 def mlstm(h, w, p, m, eps):
     t = h.shape[0]
-    H, D, V, cap = m["heads"], m["dim"], m["vdim"], m["gate_cap"]
+    H, D, V, cap = m["heads"], m["dim"], m.get("vdim") or m["dim"], m["gate_cap"]
     q = (h @ w[p + "q"].T).view(t, H, D) * D ** -0.5
     k = (h @ w[p + "k"].T).view(t, H, D)
     v = (h @ w[p + "v"].T).view(t, H, V)
@@ -193,7 +193,7 @@ def forward(cfg, weights, tokens, dtype=torch.float64, layers_out=None, margins=
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
         u = grouped_norm(x, w[p + "norm1"], groups, eps)
-        h = u + causal_conv(u, w[p + "canon1"])
+        h = u + causal_conv(u, w[p + "canon1"]) if (cfg.get("canon") or {}).get("taps") else u
         y = MIXERS[layer["type"]](h, w, p + "mix.", layer["mixer"], eps)
         x = x + y * torch.sigmoid(u @ w[p + "rg1"].T + w[p + "rg1.b"])
         mlp = layer.get("mlp")
