@@ -8,6 +8,7 @@ model with random weights (bfloat16), plus prefill throughput and roofline fract
     python bench.py --preset zudepel [--timeline]  (the Zudepel design at two sizes beside Vogilix layers of equal size)
     python bench.py --preset sozanex [--timeline]  (the Sozanex design at two sizes beside Vogilix layers of equal size)
     python bench.py --preset fasodra [--timeline]  (the Fasodra design at two sizes beside Zudepel layers of equal size)
+    python bench.py --preset midisun [--timeline]  (the Midisun design at two sizes beside Zudepel layers of equal size)
 
 Prints one JSON line. A "step" is one decode step of the whole batch (default batch 8, every
 sequence after 1,023 cached positions, context 4,096). ``value`` is decoded tokens per second
@@ -634,10 +635,27 @@ def fasodra_config(size: str, layers: int):
     return {"architecture": "Fasodra", "vocab": vocab, "width": w, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "streams": 2, "layers": out}
 
 
-def run_fasodra(args, pk, pk_source):
-    """Prefill and decode throughput of the Fasodra design at two sizes, each beside Zudepel layers of the same width, depth, heads,
-    experts and expert sizes (the library's closest model: a recurrence over a matrix state beside attention, routed experts, a
-    32-bit stream); with --timeline also the per-kernel device times of one prompt step and one decode step of both (stderr)."""
+def midisun_config(size: str, layers: int):
+    """Layers of a real model's sizes: retention, attention (capped scores, slopes, a window of 2,048), mLSTM and attention in turn; the
+    first layer dense, the others routed with groups; norms in four groups, convolutions of four taps."""
+    import math
+    w, heads, kv_heads, dim, dense, experts, groups, top, ff, vocab = {
+        "mid": (2048, 16, 4, 128, 8192, 32, (4, 2), 4, 1024, 32768),
+        "wide": (4096, 32, 8, 128, 12288, 64, (8, 4), 6, 1408, 65536)}[size]
+    moe = {"expert": {"ff": ff}, "kind": "moe", "router": {"experts": experts, "groups": {"count": groups[0], "keep": groups[1]}, "top": top}}
+    decay = [math.exp(-2.0 ** (-8.0 * (h + 1) / heads)) for h in range(heads)]
+    mixers = [("retention", {"decay": decay, "dim": dim, "heads": heads, "rot": {"base": 10000.0, "dims": dim // 2}, "vdim": dim}),
+              ("attention", {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"size": 2048}, "scale": dim ** -0.5, "softcap": 30.0, "vdim": dim}),
+              ("mlstm", {"dim": dim, "gate_cap": 15.0, "heads": heads, "vdim": dim})]
+    kinds = [mixers[(0, 1, 2, 1)[i % 4]] for i in range(layers)]
+    return {"architecture": "Midisun", "vocab": vocab, "width": w, "norm": {"eps": 1e-6, "groups": 4}, "canon": {"taps": 4}, "embedding": {"scale": 1.0},
+            "layers": [{"mixer": m, "mlp": {"ff": dense, "kind": "dense"} if i == 0 else moe, "type": t} for i, (t, m) in enumerate(kinds)]}
+
+
+def run_beside(args, pk_source, name, config, twin, twin_config):
+    """Prefill and decode throughput of a design at two sizes, each beside layers of another of the library's designs of the same width,
+    depth, heads, experts and expert sizes; with --timeline also the per-kernel device times of one prompt step and one decode step of
+    both (stderr)."""
     import torch
     from tileinfer_b200.config import config_from_dict
     from tileinfer_b200.engine import Engine
@@ -647,11 +665,11 @@ def run_fasodra(args, pk, pk_source):
     clocks.start()
     out = []
     for size in ("mid", "wide"):
-        for name, raw in (("fasodra", fasodra_config(size, layers)), ("zudepel", zudepel_config(size, layers))):
+        for model, raw in ((name, config(size, layers)), (twin, twin_config(size, layers))):
             cfg = config_from_dict(raw)
             engine = Engine.random(cfg, seed=0, dtype=args.dtype, max_context=4096, max_seqs=64, max_tokens=64 * 1280,
                                    max_step_tokens=8192)
-            row = {"size": size, "model": name, "layers": layers, "weights_gb": round(engine.weight_bytes() / 1e9, 3),
+            row = {"size": size, "model": model, "layers": layers, "weights_gb": round(engine.weight_bytes() / 1e9, 3),
                    "cache_bytes_per_position": engine.kv_bytes_per_position()}
             for tokens in (512, 2048):
                 ms = time_prefill(engine, tokens, cfg.vocab_size, reps=3)
@@ -672,14 +690,14 @@ def run_fasodra(args, pk, pk_source):
         import contextlib
         with contextlib.redirect_stdout(sys.stderr):
             for size in ("mid", "wide"):
-                for name, raw in (("fasodra", fasodra_config(size, 4)), ("zudepel", zudepel_config(size, 4))):
+                for model, raw in ((name, config(size, 4)), (twin, twin_config(size, 4))):
                     cfg = config_from_dict(raw)
-                    print(f"--- {size} {name}: prompt of 2,048 tokens")
-                    microbench.timeline(1, 0, prefill_tokens=2048, config=cfg, first=90 if name == "fasodra" else 1)
+                    print(f"--- {size} {model}: prompt of 2,048 tokens")
+                    microbench.timeline(1, 0, prefill_tokens=2048, config=cfg, first=90 if model == name else 1)
                     for b in (8, 64):
-                        print(f"--- {size} {name}: decode step of batch {b}")
-                        microbench.timeline(b, 0, config=cfg, first=90 if (b == 8 and name == "fasodra") else 1)
-    print(json.dumps({"metric": "prefill and decode of the Fasodra design beside Zudepel layers of equal size", "n_gpus": 1,
+                        print(f"--- {size} {model}: decode step of batch {b}")
+                        microbench.timeline(b, 0, config=cfg, first=90 if (b == 8 and model == name) else 1)
+    print(json.dumps({"metric": f"prefill and decode of the {name.capitalize()} design beside {twin.capitalize()} layers of equal size", "n_gpus": 1,
                       "steps": steps, "warmup": warmup, "dtype": "bf16" if args.dtype == "bfloat16" else "fp32",
                       "data": "synthetic: random weights, uniform random token ids",
                       "config": {"cached_positions": CACHED, "peaks": pk_source, "l2": "every step reads more weights than L2 holds"},
@@ -715,7 +733,7 @@ def main(argv=None) -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (quick checks)")
     ap.add_argument("--timeline", action="store_true", help="--preset vogilix: per-kernel device times of its steps, on stderr")
-    ap.add_argument("--preset", default="8b", choices=["8b", "8b-long", "70b", "sweep", "vogilix", "zudepel", "sozanex", "fasodra"],
+    ap.add_argument("--preset", default="8b", choices=["8b", "8b-long", "70b", "sweep", "vogilix", "zudepel", "sozanex", "fasodra", "midisun"],
                     help="8b: the headline line (default); 8b-long: 8 unequal sequences of up to 32,768 positions; "
                          "70b: Apertus-70B sizes, 141 GB of weights")
     args = ap.parse_args(argv)
@@ -742,7 +760,9 @@ def main(argv=None) -> int:
     if args.preset == "vogilix":
         return run_vogilix(args, *peaks())
     if args.preset == "fasodra":
-        return run_fasodra(args, *peaks())
+        return run_beside(args, peaks()[1], "fasodra", fasodra_config, "zudepel", zudepel_config)
+    if args.preset == "midisun":
+        return run_beside(args, peaks()[1], "midisun", midisun_config, "zudepel", zudepel_config)
     if args.preset == "sozanex":
         return run_sozanex(args, *peaks())
     if args.preset == "zudepel":
