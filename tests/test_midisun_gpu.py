@@ -443,16 +443,17 @@ def test_the_gates_of_the_matrix_memory_alone():
 @pytest.mark.parametrize("H,D,V", [(2, 24, 40), (1, 130, 70), (3, 64, 136), (2, 18, 14), (12, 128, 128), (1, 300, 64)])
 def test_matrix_memories_alone(H, D, V):
     """Both recurrences against loops in 64-bit, at sizes that are no multiple of a thread's rows or a block's columns: unequal sequences in
-    one launch, continued from the state by portions of 37 and 2 tokens, then one token at a time (the one-token kernel, fused with the
-    head's norm and gate where a block holds the head, and where it is not), a slot between them that nobody may touch."""
+    one launch, continued from the state by portions of 100, 37 and 2 tokens (walked one by one, and in chunks), then one token at a time
+    (the one-token kernel, fused with the head's norm and gate where a block holds the head, and where it is not), a slot between them that
+    nobody may touch."""
     from tileinfer_b200.kernels import ops
     from tileinfer_b200.parts import Runtime, lookup
     from tileinfer_b200.config import PositionSpec
     g = torch.Generator().manual_seed(D + V)
     for T in (torch.float32, torch.bfloat16):
-        lengths = [70, 1, 45]
+        lengths = [150, 1, 145]
         n = sum(lengths)
-        rot = min(D, 16)
+        rot = 16 if D != 300 else 290
         rotation = lookup("position", "rope")(PositionSpec("rope", D, 100.0, None, 256, {"rotary_dim": rot, "table_dtype": "float32", "angles": "float64"}),
                                               Runtime(T), 256).rotation()
         proj = rnd(torch.randn(n, H * (2 * D + 2 * V), generator=g, dtype=F64) * 0.6, T)
@@ -483,55 +484,65 @@ def test_matrix_memories_alone(H, D, V):
                         o[t] = torch.einsum("hdv,hd->hv", S, qr[t])
                     ref[at:at + L] = plain.rms_divide(o, eps).reshape(L, -1) * plain.silu(gate)
                 at += L
-            floats = -(-(H * D * V + (H * (D + 1) if gated else 0)) // 4) * 4
-            state = torch.zeros(4, floats, device="cuda")
-            m_off = H * D * (V + 1)
-            dev = lambda t, dt=torch.float32: t.to(dt).cuda().contiguous()
-            starts, fed, slots = [0, 70, 71], [0, 0, 0], [2, 0, 3]
-            got = torch.zeros(n, H * V, dtype=F64)
-            for portion in (37, 2) + (1,) * 40:
-                live = [b for b in range(3) if fed[b] < lengths[b]]
-                if not live:
-                    break
-                take = [min(portion, lengths[b] - fed[b]) for b in live]
-                idx = torch.cat([torch.arange(starts[b] + fed[b], starts[b] + fed[b] + c) for b, c in zip(live, take)])
-                pos = [fed[b] + j for b, c in zip(live, take) for j in range(c)]
-                step = _step(take, [slots[b] for b in live], pos)
-                rows_, zz = dev(proj[idx], T), dev(z[idx])
-                y = torch.full((len(idx), H * V), float("nan"), dtype=T, device="cuda")
-                o = torch.full((len(idx), H * V), float("nan"), device="cuda")
-                nq, em, mn = (torch.full((len(idx), H), float("nan"), device="cuda") for _ in range(3))
-                cell = dict(z=zz, bias=dev(bias), cap=cap, q_scale=D ** -0.5, w=dev(norm_w, T), gate_sigmoid=True) if gated else \
-                    dict(decay=dev(decay), rotation=rotation, k_scale=D ** -0.5)
-                divisor, moves, done = ((nq, em) if gated else None), None, False
-                if all(c == 1 for c in take):
-                    if V <= 128 and len(live) % 2:                                   # fused, or raw and finished by the norm's kernel
-                        done = ops.memory_token(rows_, offs, state, step, H, D, V, y=y, eps=eps, **cell)
-                        fused = done
+            for chunked in (False, True):
+                floats = -(-(H * D * V + (H * (D + 1) if gated else 0)) // 4) * 4
+                state = torch.zeros(4, floats, device="cuda")
+                m_off = H * D * (V + 1)
+                dev = lambda t, dt=torch.float32: t.to(dt).cuda().contiguous()
+                starts, fed, slots = [0, 150, 151], [0, 0, 0], [2, 0, 3]
+                got = torch.zeros(n, H * V, dtype=F64)
+                for portion in (100, 37, 2) + (1,) * 40:
+                    live = [b for b in range(3) if fed[b] < lengths[b]]
+                    if not live:
+                        break
+                    take = [min(portion, lengths[b] - fed[b]) for b in live]
+                    idx = torch.cat([torch.arange(starts[b] + fed[b], starts[b] + fed[b] + c) for b, c in zip(live, take)])
+                    pos = [fed[b] + j for b, c in zip(live, take) for j in range(c)]
+                    step = _step(take, [slots[b] for b in live], pos)
+                    rows_, zz = dev(proj[idx], T), dev(z[idx])
+                    y = torch.full((len(idx), H * V), float("nan"), dtype=T, device="cuda")
+                    o = torch.full((len(idx), H * V), float("nan"), device="cuda")
+                    nq, em, mn = (torch.full((len(idx), H), float("nan"), device="cuda") for _ in range(3))
+                    cell = dict(z=zz, bias=dev(bias), cap=cap, q_scale=D ** -0.5, w=dev(norm_w, T), gate_sigmoid=True) if gated else \
+                        dict(decay=dev(decay), rotation=rotation, k_scale=D ** -0.5)
+                    divisor, moves, done = ((nq, em) if gated else None), None, False
+                    if all(c == 1 for c in take):
+                        if V <= 128 and len(live) % 2:                                   # fused, or raw and finished by the norm's kernel
+                            done = ops.memory_token(rows_, offs, state, step, H, D, V, y=y, eps=eps, **cell)
+                            fused = done
+                        else:
+                            done = ops.memory_token(rows_, offs, state, step, H, D, V, o=o, outs=(nq, em, mn) if gated else (None,) * 3, **cell)
+                            fused = False
+                            moves = (mn, state[:, m_off:m_off + H], step.seq_slots) if gated else None
+                        assert done == (V % 4 == 0)
+                        moves = moves if done else None
                     else:
-                        done = ops.memory_token(rows_, offs, state, step, H, D, V, o=o, outs=(nq, em, mn) if gated else (None,) * 3, **cell)
                         fused = False
-                        moves = (mn, state[:, m_off:m_off + H], step.seq_slots) if gated else None
-                    assert done == (V % 4 == 0)
-                    moves = moves if done else None
-                else:
-                    fused = False
-                if not done:
-                    if gated:
-                        coef = torch.zeros(len(idx), H, 2, device="cuda")
-                        ops.memory_gates(coef, em, zz, dev(bias), cap, state, m_off, step, H)
-                        ops.memory_scan(o, nq, rows_, *offs[:3], state, coef, D ** -0.5, 1.0, step, H, D, V)
-                    else:
-                        ops.retention_scan(o, rows_, *offs[:3], state, dev(decay), rotation, 1.0, D ** -0.5, step, H, D, V)
-                if not fused:
-                    ops.heads_norm_gate(y, o, rows_[:, offs[3]:], dev(norm_w, T) if gated else None, eps, H, V, gate_sigmoid=gated, divisor=divisor, moves=moves)
-                got[idx] = y.cpu().double()
-                for b, c in zip(live, take):
-                    fed[b] += c
-            err = (got - ref).abs().max(-1).values
-            tol = (1e-4 if T == torch.float32 else 2.0 ** -7) * max(1.0, float(ref.abs().max()))
-            assert float(err.max()) <= tol, f"{T} gated {gated} {H} heads {D} x {V}: {float(err.max()):.3g} at {int(err.argmax())}"
-            assert float(state[1].abs().max()) == 0.0
+                    if not done and chunked and max(take) > 1:
+                        chunks, floats_ws = ops.memory_chunk_sizes(take, H, D, V)
+                        ws, tot = torch.full((floats_ws,), float("nan"), device="cuda"), torch.full((chunks, H), float("nan"), device="cuda")
+                        kw = dict(k_scale=D ** -0.5, decay=dev(decay), rotation=rotation)
+                        if gated:
+                            kw = dict(q_scale=D ** -0.5, coef=torch.zeros(len(idx), H, 2, device="cuda"), em=em, w=dev(norm_w, T), gate_sigmoid=True)
+                            ops.memory_gates(kw["coef"], em, zz, dev(bias), cap, state, m_off, step, H)
+                        fused = V <= 128
+                        ops.memory_chunks(rows_, offs, state, step, H, D, V, ws, tot, chunks, y=y if fused else None, o=None if fused else o, nq=nq, eps=eps, **kw)
+                    elif not done:
+                        if gated:
+                            coef = torch.zeros(len(idx), H, 2, device="cuda")
+                            ops.memory_gates(coef, em, zz, dev(bias), cap, state, m_off, step, H)
+                            ops.memory_scan(o, nq, rows_, *offs[:3], state, coef, D ** -0.5, 1.0, step, H, D, V)
+                        else:
+                            ops.retention_scan(o, rows_, *offs[:3], state, dev(decay), rotation, 1.0, D ** -0.5, step, H, D, V)
+                    if not fused:
+                        ops.heads_norm_gate(y, o, rows_[:, offs[3]:], dev(norm_w, T) if gated else None, eps, H, V, gate_sigmoid=gated, divisor=divisor, moves=moves)
+                    got[idx] = y.cpu().double()
+                    for b, c in zip(live, take):
+                        fed[b] += c
+                err = (got - ref).abs().max(-1).values
+                tol = (1e-4 if T == torch.float32 else 2.0 ** -7) * max(1.0, float(ref.abs().max()))
+                assert float(err.max()) <= tol, f"{T} gated {gated} chunked {chunked} {H} heads {D} x {V}: {float(err.max()):.3g} at {int(err.argmax())}"
+                assert float(state[1].abs().max()) == 0.0
 
 
 @pytest.mark.parametrize("dtype", sorted(DTYPES))
@@ -738,7 +749,7 @@ def test_bfloat16_steps_take_the_fast_kernels(models):
     engine.free_sequence(slot)
     engine.check_health()
     assert prompt.get("ti_attention_prefill_tc_ruled", 0) == 2 and token.get("ti_attention_decode_ruled", 0) == 2, (prompt, token)
-    assert prompt.get("ti_retention_scan", 0) == 2 and prompt.get("ti_memory_scan", 0) == 2 and prompt.get("ti_conv_rows", 0) == 6, prompt
+    assert prompt.get("ti_memory_chunks", 0) == 4 and prompt.get("ti_memory_gates", 0) == 2 and prompt.get("ti_conv_rows", 0) == 6, prompt
     assert token.get("ti_memory_token", 0) == 4 and token.get("ti_heads_norm_gate", 0) == 2 and "ti_conv_rows" not in token, token
     for used in (prompt, token):
         assert used.get("ti_gemm_tcgen05_grouped", 0) == 8 and used.get("ti_gated_add_norm32", 0) == 13, used

@@ -90,6 +90,9 @@ _SIGNATURES = {
 }
 
 
+_KERNELS_PER_CALL = {"ti_memory_chunks": 3}
+
+
 def lib():
     """The loaded library (built at the first call if the sources changed)."""
     global _lib
@@ -117,12 +120,14 @@ def lib():
     wrapped.ti_gemm_tcgen05_decode_plan = handle.ti_gemm_tcgen05_decode_plan
     handle.ti_expert_plan_max_tiles.restype, handle.ti_expert_plan_max_tiles.argtypes = c_int, [c_int, c_int, c_int]
     wrapped.ti_expert_plan_max_tiles = handle.ti_expert_plan_max_tiles
+    handle.ti_memory_chunk_pitch.restype, handle.ti_memory_chunk_pitch.argtypes = c_int, [c_int, c_int]
+    wrapped.ti_memory_chunk_pitch = handle.ti_memory_chunk_pitch
     wrapped.handle = handle
     for name, args in _SIGNATURES.items():
         fn = getattr(handle, name)
         fn.restype = c_int
         fn.argtypes = args
-        setattr(wrapped, name, _Counted(fn, name))
+        setattr(wrapped, name, _Counted(fn, name, _KERNELS_PER_CALL.get(name, 1)))
     _lib = wrapped
     return wrapped
 
@@ -234,6 +239,7 @@ _SIGNATURES.update({
     "ti_retention_scan": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _I, _P, _F, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "ti_memory_gates": [_P, _P, _P, _L, _P, _F, _P, _L, _P, _P, _I, _I, _P],
     "ti_memory_scan": [_P, _P, _P, _L, _I, _I, _I, _P, _L, _P, _F, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ti_memory_chunks": [_P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P, _L, _P, _P, _P, _I, _P, _F, _F, _P, _I, _F, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     "ti_memory_token": [_P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P, _L, _P, _P, _L, _P, _F, _P, _I, _P, _F, _F, _P, _I, _F, _P, _I, _I, _I, _I,
                         _I, _P],
 })

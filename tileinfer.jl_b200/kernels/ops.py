@@ -822,3 +822,27 @@ def memory_token(rows, offs, state, step, heads, dim, vdim, y=None, o=None, outs
         return False
     check(rc, "memory_token")
     return True
+
+
+CHUNK_TOKENS = 64           # tokens of a chunk (csrc/memory_chunks.cu)
+
+
+def memory_chunk_sizes(q_lens, heads, dim, vdim):
+    """(chunks of a step with these new tokens per sequence, floats of its work space)."""
+    chunks = sum(-(-n // CHUNK_TOKENS) for n in q_lens)
+    return chunks, chunks * heads * int(lib().ti_memory_chunk_pitch(dim, vdim))
+
+
+def memory_chunks(rows, offs, state, step, heads, dim, vdim, ws, total, chunks, y=None, o=None, nq=None, em=None, decay=None, coef=None, rotation=None,
+                  q_scale=1.0, k_scale=1.0, w=None, gate_sigmoid=False, eps=1e-6):
+    """A step's tokens of retention (``decay``) or of the gated cell (``coef``, ``em`` of ``memory_gates``) in chunks: ``y`` the normed and
+    gated heads (value sizes up to 128), or ``o`` (and ``nq``) the raw ones. ``ws``, ``total`` [chunks, heads]: float32 work space."""
+    for t, name in ((state, "state"), (ws, "ws"), (total, "total")):
+        _need(t, name, torch.float32, contiguous=False)
+    _need(rows, "rows", contiguous=False)
+    if ws.numel() < chunks * heads * int(lib().ti_memory_chunk_pitch(dim, vdim)) or total.numel() < chunks * heads:
+        raise KernelError(f"memory_chunks: work space of {ws.numel()} floats for {chunks} chunks")
+    check(lib().ti_memory_chunks(_ptr(y), _ptr(o), _ptr(nq), _ptr(em), rows.data_ptr(), rows.stride(0), *offs, state.data_ptr(), state.stride(0), _ptr(decay),
+                                 _ptr(coef), *_rotation_args(rotation, step), q_scale, k_scale, _ptr(w), int(bool(gate_sigmoid)), eps, ws.data_ptr(),
+                                 total.data_ptr(), chunks, step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), step.n_seqs, heads, dim, vdim,
+                                 dtype_code(rows.dtype), _stream()), "memory_chunks")

@@ -18,8 +18,9 @@ past and of the new token are one number each per head, fixed or from the token.
 Each asks the cache for one state of floats per sequence: S, and for mlstm n and m behind it. State, rotation, gates, divisor and norm are
 32-bit in every element type; the four projections of a layer are one product (rounded to the model's element type), the gates' logits a
 second one whose sums are not rounded. A step of one token per sequence is one kernel from the projections to the output projection's
-input (``csrc/matrix_memory.cu``; heads of more than 128 values and sizes it refuses take two to four); other steps scan the step's
-tokens (``csrc/lightning_scan.cuh``).
+input (``csrc/matrix_memory.cu``; heads of more than 128 values and sizes it refuses take two to four). Steps that bring a sequence
+CHUNKED_FROM tokens or more cut its tokens into chunks that are worked on side by side (``csrc/memory_chunks.cu``), other steps scan their
+tokens one by one (``csrc/lightning_scan.cuh``).
 
 Record: ``num_heads``, ``head_dim`` (query/key size) and the options ``value_dim``, ``norm_eps``; retention: ``decay`` (one number per
 head) and the position encoding's rotation, if any; mlstm: ``gate_cap``.
@@ -33,15 +34,14 @@ from ..kernels import ops
 from .base import CacheRequest, Mixer, register_mixer
 from .linear import Linear
 
-FUSED_VALUES = 128          # value sizes up to which a block of the one-token kernel holds a whole head
+FUSED_VALUES = 128          # value sizes up to which a block of the one-token and of the chunked kernels holds a whole head
+CHUNKED_FROM = 96           # new tokens of a step's longest sequence from which on its tokens are worked on in chunks
 
 
 class MatrixMemory(Mixer):
-    """What the two cells share. A cell sets ``q_scale``, ``k_scale``, ``norm_w``, ``gate_sigmoid``, ``vector`` (whether n and m lie behind
-    S) and offers ``token`` and ``scan``."""
-    name, vector, gate_sigmoid = "", False, False
-    norm_w = None
-    q_scale = k_scale = 1.0
+    """What the two cells share. A cell sets ``name``, ``vector`` (whether n and m lie behind S) and ``constants`` (the scales of q and k, the
+    rotation, the weight and gate of the heads' norm, and retention's decays)."""
+    name, vector = "", False
 
     def __init__(self, spec: MixerSpec, tensors, rt, position):
         self.spec, self.rt = spec, rt
@@ -66,18 +66,47 @@ class MatrixMemory(Mixer):
         floats = self.heads * self.dim * self.vdim + (self.heads * (self.dim + 1) if self.vector else 0)
         return CacheRequest("state", shape=(-(-floats // 4) * 4,), dtype=torch.float32)          # whole 16-byte pieces per sequence
 
+    def gate_logits(self, h):
+        """The gates' logits [n, 2 heads] in 32-bit, or None."""
+        return None
+
     def forward(self, h, step, cache):
-        rt = self.rt
-        n, H, V = h.shape[0], self.heads, self.vdim
-        rows = rt.buffer(self.name + ".rows", (n, self.proj.out_features))
-        self.proj.forward(h, rows)
+        rt, c = self.rt, self.constants
+        n, H, D, V = h.shape[0], self.heads, self.dim, self.vdim
+        state, sizes = cache.state, (self.heads, self.dim, self.vdim)
+        rows = self.proj.forward(h, rt.buffer(self.name + ".rows", (n, self.proj.out_features)))
+        z = self.gate_logits(h)
         y = rt.buffer(self.name + ".normed", (n, H * V))
-        if not (step.is_decode and self.token(h, rows, y, step, cache.state)):
-            o = rt.buffer(self.name + ".o", (n, H * V), torch.float32)
-            divisor, moves = self.scan(h, rows, o, step, cache.state)
-            ops.heads_norm_gate(y, o, rows[:, self.offs[3]:], self.norm_w, self.eps, H, V, gate_sigmoid=self.gate_sigmoid, divisor=divisor, moves=moves)
-        out = rt.buffer("mixer.delta", (n, self.spec.hidden_size))
-        return self.o.forward(y, out, allow_partials=True)
+        fused = V <= FUSED_VALUES
+        # Where a block holds a whole head it leaves y; else the raw heads o (with the gated cell's divisor) go through the norm's kernel.
+        o = None if fused else rt.buffer(self.name + ".o", (n, H * V), torch.float32)
+        nq, em, m_new = (rt.buffer(f"{self.name}.{k}", (n, H), torch.float32) for k in ("nq", "em", "m_new")) if self.vector else (None, None, None)
+        where = dict(y=y if fused else None, o=o, q_scale=c["q_scale"], k_scale=c["k_scale"], rotation=c["rotation"], w=c["w"],
+                     gate_sigmoid=c["gate_sigmoid"], eps=self.eps, decay=c["decay"])
+        moves = None
+        if step.is_decode and ops.memory_token(rows, self.offs, state, step, *sizes, outs=(None,) * 3 if fused else (nq, em, m_new), z=z,
+                                               bias=c["gate_bias"], cap=c["gate_cap"], **where):
+            if self.vector and not fused:
+                moves = (m_new, state[:, self.m_off:self.m_off + H], step.seq_slots)
+        else:
+            coef = None
+            if self.vector:
+                coef = rt.buffer(self.name + ".coef", (n, H, 2), torch.float32)
+                ops.memory_gates(coef, em, z, c["gate_bias"], c["gate_cap"], state, self.m_off, step, H)
+            if step.max_q_len >= CHUNKED_FROM:
+                chunks, floats = ops.memory_chunk_sizes(step.host_q_lens, *sizes)
+                ws, total = rt.buffer("memory.chunks", (floats,), torch.float32), rt.buffer("memory.totals", (chunks, H), torch.float32)
+                ops.memory_chunks(rows, self.offs, state, step, *sizes, ws, total, chunks, nq=nq, em=em, coef=coef, **where)
+            else:
+                fused, o = False, rt.buffer(self.name + ".o", (n, H * V), torch.float32)
+                if self.vector:
+                    ops.memory_scan(o, nq, rows, *self.offs[:3], state, coef, c["q_scale"], c["k_scale"], step, *sizes)
+                else:
+                    ops.retention_scan(o, rows, *self.offs[:3], state, c["decay"], c["rotation"], c["q_scale"], c["k_scale"], step, *sizes)
+        if not fused:
+            ops.heads_norm_gate(y, o, rows[:, self.offs[3]:], c["w"], self.eps, H, V, gate_sigmoid=c["gate_sigmoid"],
+                                divisor=(nq, em) if self.vector else None, moves=moves)
+        return self.o.forward(y, rt.buffer("mixer.delta", (n, self.spec.hidden_size)), allow_partials=True)
 
 
 @register_mixer("retention")
@@ -89,36 +118,22 @@ class Retention(MatrixMemory):
         decay = [float(a) for a in spec.options["decay"]]
         if len(decay) != self.heads:
             raise ValueError(f"retention: {len(decay)} decays for {self.heads} heads")
-        self.decay = torch.tensor(decay, dtype=torch.float64).float().to(rt.device)
-        self.k_scale = self.dim ** -0.5
-        self.rotation = position.rotation() if position is not None else None
-
-    def token(self, h, rows, y, step, state):
-        return self.vdim <= FUSED_VALUES and ops.memory_token(rows, self.offs, state, step, self.heads, self.dim, self.vdim, y=y, decay=self.decay,
-                                                              rotation=self.rotation, k_scale=self.k_scale, eps=self.eps)
-
-    def scan(self, h, rows, o, step, state):
-        done = step.is_decode and ops.memory_token(rows, self.offs, state, step, self.heads, self.dim, self.vdim, o=o, decay=self.decay,
-                                                   rotation=self.rotation, k_scale=self.k_scale)
-        if not done:
-            ops.retention_scan(o, rows, *self.offs[:3], state, self.decay, self.rotation, 1.0, self.k_scale, step, self.heads, self.dim, self.vdim)
-        return None, None
+        self.constants = {"q_scale": 1.0, "k_scale": self.dim ** -0.5, "rotation": position.rotation() if position is not None else None, "w": None,
+                          "gate_sigmoid": False, "decay": torch.tensor(decay, dtype=torch.float64).float().to(rt.device), "gate_bias": None, "gate_cap": 0.0}
 
 
 @register_mixer("mlstm")
 class MLstm(MatrixMemory):
-    name, vector, gate_sigmoid = "mlstm", True, True
+    name, vector = "mlstm", True
 
     def __init__(self, spec: MixerSpec, tensors, rt, position):
         super().__init__(spec, tensors, rt, position)
         n, p = spec.tensor_names, spec.prefix
-        self.cap = float(spec.options["gate_cap"])
-        self.q_scale = self.dim ** -0.5
-        self.norm_w = rt.param(tensors[p + n["norm"]])
         self.gates = Linear(torch.cat([rt.param(tensors[p + n[k]]) for k in ("i", "f")], 0).contiguous(), rt, "mlstm_gates")
         bias = [rt.param(tensors[p + n[k] + n["bias_suffix"]], keep_dtype=True).float().flatten() for k in ("i", "f")]
-        self.gate_bias = torch.cat(bias).contiguous()
         self.m_off = self.heads * self.dim * (self.vdim + 1)             # where m lies in a sequence's state, behind S and n
+        self.constants = {"q_scale": self.dim ** -0.5, "k_scale": 1.0, "rotation": None, "w": rt.param(tensors[p + n["norm"]]), "gate_sigmoid": True,
+                          "decay": None, "gate_bias": torch.cat(bias).contiguous(), "gate_cap": float(spec.options["gate_cap"])}
 
     @classmethod
     def tensors(cls, spec: MixerSpec):
@@ -130,23 +145,5 @@ class MLstm(MatrixMemory):
                     TensorDecl(p + n[k] + n["bias_suffix"], (H,), ("const_plus_normal", mean, 1.0), keep_dtype=True)]
         return out
 
-    def _logits(self, h):
+    def gate_logits(self, h):
         return self.gates.forward_f32(h, self.rt.buffer("mlstm.gates", (h.shape[0], 2 * self.heads), torch.float32))
-
-    def _token(self, h, rows, step, state, **where):
-        return ops.memory_token(rows, self.offs, state, step, self.heads, self.dim, self.vdim, z=self._logits(h), bias=self.gate_bias, cap=self.cap,
-                                q_scale=self.q_scale, w=self.norm_w, gate_sigmoid=True, eps=self.eps, **where)
-
-    def token(self, h, rows, y, step, state):
-        return self.vdim <= FUSED_VALUES and self._token(h, rows, step, state, y=y)
-
-    def scan(self, h, rows, o, step, state):
-        rt, H, n = self.rt, self.heads, h.shape[0]
-        nq, em, m_new = (rt.buffer("mlstm." + k, (n, H), torch.float32) for k in ("nq", "em", "m_new"))
-        m = state[:, self.m_off:self.m_off + H]
-        if step.is_decode and self._token(h, rows, step, state, o=o, outs=(nq, em, m_new)):
-            return (nq, em), (m_new, m, step.seq_slots)
-        coef = rt.buffer("mlstm.coef", (n, H, 2), torch.float32)
-        ops.memory_gates(coef, em, self._logits(h), self.gate_bias, self.cap, state, self.m_off, step, H)
-        ops.memory_scan(o, nq, rows, *self.offs[:3], state, coef, self.q_scale, 1.0, step, H, self.dim, self.vdim)
-        return (nq, em), None
