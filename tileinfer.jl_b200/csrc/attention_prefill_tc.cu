@@ -79,6 +79,50 @@ __device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
     asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
     return d;
 }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+// A row's scores r (unscaled) capped, in base-2 units: cap log2(e) tanh(x), x = scale r / cap. Where no row of the warp has |x| > 1/2 the
+// odd series of tanh to its seventh term (the rest is below 1e-7 of x there) does it on the FMA units, two lanes an instruction, which
+// leaves the exponential unit to the softmax; else the closed form.
+__device__ __forceinline__ void cap_row(unsigned (&r)[4][32], const AttnExtras& ex, float scale_log2) {
+    float top[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) top[i & 3] = fmaxf(top[i & 3], fabsf(__uint_as_float(r[c][i])));
+    if (__all_sync(0xffffffffu, fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) <= ex.cap_small)) {
+        // tanh x / x = sum_n a_n (x^2)^n with a_n from the Bernoulli numbers; the powers of (scale / cap)^2 are folded in.
+        const float u = ex.cap_ratio2, u2 = u * u, u4 = u2 * u2;
+        const f32x2 one = pack2(1.f, 1.f), s2 = pack2(scale_log2, scale_log2);
+        const float a1 = -u / 3.f, a2 = u2 * (2.f / 15.f), a3 = u2 * u * (-17.f / 315.f), a4 = u4 * (62.f / 2835.f), a5 = u4 * u * (-1382.f / 155925.f),
+                    a6 = u4 * u2 * (21844.f / 6081075.f);
+        const f32x2 b1 = pack2(a1, a1), b2 = pack2(a2, a2), b3 = pack2(a3, a3), b4 = pack2(a4, a4), b5 = pack2(a5, a5), b6 = pack2(a6, a6);
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+                const f32x2 x = pack2(__uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1])), y = mul2(x, x);
+                f32x2 p = fma2(b6, y, b5);
+                p = fma2(p, y, b4);
+                p = fma2(p, y, b3);
+                p = fma2(p, y, b2);
+                p = fma2(p, y, b1);
+                p = fma2(p, y, one);
+                float v0, v1;
+                unpack2(mul2(mul2(x, s2), p), v0, v1);
+                r[c][i] = __float_as_uint(v0);
+                r[c][i + 1] = __float_as_uint(v1);
+            }
+        return;
+    }
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) r[c][i] = __float_as_uint(capped_score2(__uint_as_float(r[c][i]), ex));
+}
 template <int D>
 __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                           const __grid_constant__ CUtensorMap map_k,
@@ -123,6 +167,10 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
     if (p.ex.chunk > 0) key_lo = max(key_lo, ((start + t0) / p.ex.chunk) * p.ex.chunk);        // the chunk of the block's first token
     const int j_lo = key_lo / KEYS, j_hi = (key_hi + KEYS - 1) / KEYS;
     const int n_pages = (kv_len + PAGE - 1) / PAGE;
+    // With a slope by distance the nearest keys come first: a row's largest scores are then among the first it meets, and its output does
+    // not have to be rescaled from tile to tile.
+    const bool backward = p.ex.slope != nullptr;
+    auto tile_of = [&](int j) { return backward ? j_hi - 1 - (j - j_lo) : j; };
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -160,13 +208,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
             // what stands in shared memory must be finite.
             const int* table = p.table + (long long)slot * p.table_stride;
             int page[KEYS / PAGE], next_page[KEYS / PAGE];
-            for (int pg = 0; pg < KEYS / PAGE; ++pg) page[pg] = __ldcg(table + min(j_lo * (KEYS / PAGE) + pg, n_pages - 1));
+            for (int pg = 0; pg < KEYS / PAGE; ++pg) page[pg] = __ldcg(table + min(tile_of(j_lo) * (KEYS / PAGE) + pg, n_pages - 1));
             bool ok = true;
             int fill = 0;                                       // K_j is fill 2(j - j_lo), V_j the next one
             for (int j = j_lo; ok && j < j_hi; ++j) {
                 // The next step's page numbers are on their way while this step's tiles are waited for.
                 for (int pg = 0; pg < KEYS / PAGE; ++pg)
-                    next_page[pg] = j + 1 < j_hi ? __ldcg(table + min((j + 1) * (KEYS / PAGE) + pg, n_pages - 1)) : 0;
+                    next_page[pg] = j + 1 < j_hi ? __ldcg(table + min(tile_of(j + 1) * (KEYS / PAGE) + pg, n_pages - 1)) : 0;
                 for (int kv = 0; kv < 2; ++kv, ++fill) {
                     const int buf = fill % RING;
                     const unsigned phase = (unsigned)(fill / RING) & 1u;
@@ -257,7 +305,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
             ok = __all_sync(0xffffffffu, mbar_wait(s_full0 + 8 * x, jphase, p.status, 7));
             if (!ok) break;
             tc_fence_after();
-            const int key0 = j * KEYS;
+            const int key0 = tile_of(j) * KEYS;
             // Warp-uniform: does any row of this warp have a masked key in this step?
             const bool masked = key0 + KEYS - 1 > warp_pos_lo || (p.window > 0 && key0 <= warp_pos_hi - p.window) ||
                                 (p.ex.chunk > 0 && key0 < (warp_pos_hi / p.ex.chunk) * p.ex.chunk);
@@ -269,14 +317,21 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
 #pragma unroll
             for (int c = 0; c < 4; ++c) tmem_ld32(s_addr + c * 32, r[c]);
             tmem_ld_wait();
-            if (p.ex.cap_out > 0.f || p.ex.slope != nullptr) {
+            if (p.ex.cap_out > 0.f) cap_row(r, p.ex, p.scale_log2);
+            float row_base = 0.f;                               // what every score of the tile still lacks
+            if (p.ex.slope != nullptr) {
+                const float by = p.ex.cap_out > 0.f ? 1.0f : p.scale_log2;
+                row_base = slope * (float)(key0 - pos);
 #pragma unroll
                 for (int c = 0; c < 4; ++c)
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) {
-                        const float raw = __uint_as_float(r[c][i]);
-                        const float s = p.ex.cap_out > 0.f ? capped_score2(raw, p.ex) : raw * p.scale_log2;
-                        r[c][i] = __float_as_uint(fmaf(slope, (float)(key0 + c * 32 + i - pos), s));
+                    for (int i = 0; i < 32; i += 2) {
+                        const f32x2 x2 = fma2(pack2(__uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1])), pack2(by, by),
+                                              mul2(pack2(slope, slope), pack2((float)(c * 32 + i), (float)(c * 32 + i + 1))));
+                        float v0, v1;
+                        unpack2(x2, v0, v1);
+                        r[c][i] = __float_as_uint(v0);
+                        r[c][i + 1] = __float_as_uint(v1);
                     }
             }
             const float bias_scale = p.ex.cap_out > 0.f || p.ex.slope != nullptr ? 1.0f : p.scale_log2;
@@ -307,7 +362,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
 #pragma unroll
                 for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(r[c][i]));
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const float mt = fmaxf(mx * score_scale, -1e30f);
+            const float mt = fmaxf(fmaf(mx, score_scale, row_base), -1e30f);
             if (j == j_lo) {
                 m_used = mt;
             } else if (__any_sync(0xffffffffu, mt > m_used + RESCALE_STEP)) {
@@ -331,7 +386,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
                 tmem_st_wait();
             }
             f32x2 l2[2] = {0ull, 0ull};                          // two chains of packed sums
-            const f32x2 scale2 = pack2(score_scale, score_scale), neg_m2 = pack2(-m_used, -m_used);
+            const f32x2 scale2 = pack2(score_scale, score_scale), neg_m2 = pack2(row_base - m_used, row_base - m_used);
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
                 unsigned packed[16];

@@ -224,11 +224,14 @@ struct AttnExtras {
     const float* bias;
     int bias_len;
     float cap_in = 0.f, cap_out = 0.f;
+    float cap_small = 0.f;               // scores (unscaled) up to which |scale * score / cap| <= 1/2
+    float cap_ratio2 = 0.f;              // (scale / cap)^2
     const float* slope = nullptr;
 };
 inline AttnExtras attn_extras(int chunk, const float* bias, int bias_len, float scale, float cap, const float* slope) {
     AttnExtras ex = {chunk, bias, bias_len};
     if (cap > 0.f) { ex.cap_in = 2.f * scale * 1.4426950408889634f / cap; ex.cap_out = cap * 1.4426950408889634f; }
+    if (cap > 0.f && scale != 0.f) { ex.cap_small = 0.5f * cap / (scale < 0.f ? -scale : scale); ex.cap_ratio2 = (scale / cap) * (scale / cap); }
     ex.slope = slope;
     return ex;
 }

@@ -206,12 +206,19 @@ extern "C" int ti_gated_add_norm32(float* x, const void* d, const float* d_parti
 }
 
 // ------------------------------------------------------------------------------------------------ the convolution over a step's rows
-#define CR_TOKENS 8
-template <typename T, int VEC>
+#define CR_TOKENS 16
+// A thread owns VEC channels and walks a few rows; with the number of taps known at compile time (TAPS > 0) the rows before the current
+// one stay in registers. A row's sum is taken in the order of the taps either way.
+template <typename T, int VEC, int TAPS>
 __global__ void conv_rows_kernel(T* __restrict__ out, const T* h, const T* __restrict__ conv, int taps, const float* hist, long long hist_stride,
                                  const int* cu_seqlens, const int* seq_slots, int B, int n, int size) {
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     const int first = blockIdx.y * CR_TOKENS, last = min(n, first + CR_TOKENS);
+    constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0;
+    float c[TAPS > 0 ? TAPS : 1][VEC], w[BACK > 0 ? BACK : 1][VEC];          // weights; the rows before the current one, oldest first
+    if (TAPS > 0 && i < size)
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) Piece<T, VEC>::load(conv + (size_t)j * size + i, c[j]);
     pdl_enter();
     if (i >= size) return;
     int lo = 0, hi = B - 1;                              // the sequence of the first row: the last b with cu[b] <= first
@@ -220,23 +227,48 @@ __global__ void conv_rows_kernel(T* __restrict__ out, const T* h, const T* __res
         if (__ldcg(cu_seqlens + mid) <= first) lo = mid; else hi = mid - 1;
     }
     int b = lo, begin = __ldcg(cu_seqlens + b), end = __ldcg(cu_seqlens + b + 1);
+    auto earlier = [&](int r, float (&u)[VEC]) {         // row r of the step, or, ahead of the sequence's first, a row of its history
+        if (r >= begin) Piece<T, VEC>::load(h + (size_t)r * size + i, u);
+        else Piece<float, VEC>::load(hist + (size_t)__ldcg(seq_slots + b) * hist_stride + (size_t)(taps - 1 + r - begin) * size + i, u);
+    };
+    bool fresh = true;
     for (int t = first; t < last; ++t) {
-        while (t >= end) { ++b; begin = end; end = __ldcg(cu_seqlens + b + 1); }
-        float acc[VEC], u[VEC], c[VEC], v[VEC];
+        while (t >= end) { ++b; begin = end; end = __ldcg(cu_seqlens + b + 1); fresh = true; }
+        float acc[VEC], v[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
-        for (int j = 0; j < taps - 1; ++j) {
-            const int r = t - (taps - 1) + j;
-            if (r >= begin) Piece<T, VEC>::load(h + (size_t)r * size + i, u);
-            else Piece<float, VEC>::load(hist + (size_t)__ldcg(seq_slots + b) * hist_stride + (size_t)(taps - 1 + r - begin) * size + i, u);
-            Piece<T, VEC>::load(conv + (size_t)j * size + i, c);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) acc[e] = fmaf(c[e], u[e], acc[e]);
-        }
         Piece<T, VEC>::load(h + (size_t)t * size + i, v);
-        Piece<T, VEC>::load(conv + (size_t)(taps - 1) * size + i, c);
+        if constexpr (TAPS > 0) {
+            if (fresh) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] = v[e] + fmaf(c[e], v[e], acc[e]);
+                for (int j = 0; j < BACK; ++j) earlier(t - BACK + j, w[j]);
+                fresh = false;
+            }
+#pragma unroll
+            for (int j = 0; j < BACK; ++j)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) acc[e] = fmaf(c[j][e], w[j][e], acc[e]);
+#pragma unroll
+            for (int j = 0; j + 1 < BACK; ++j)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) w[j][e] = w[j + 1][e];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                if (BACK > 0) w[BACK > 0 ? BACK - 1 : 0][e] = v[e];
+                acc[e] = v[e] + fmaf(c[BACK][e], v[e], acc[e]);
+            }
+        } else {
+            float u[VEC], k[VEC];
+            for (int j = 0; j < taps - 1; ++j) {
+                earlier(t - (taps - 1) + j, u);
+                Piece<T, VEC>::load(conv + (size_t)j * size + i, k);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) acc[e] = fmaf(k[e], u[e], acc[e]);
+            }
+            Piece<T, VEC>::load(conv + (size_t)(taps - 1) * size + i, k);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] = v[e] + fmaf(k[e], v[e], acc[e]);
+        }
         Piece<T, VEC>::store(out + (size_t)t * size + i, acc);
     }
 }
@@ -246,13 +278,24 @@ extern "C" int ti_conv_rows(void* out, const void* h, const void* conv, int taps
                             const int* seq_slots, int n, int B, int size, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
     TI_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS && (taps == 1 || hist != nullptr) && B >= 1, "conv_rows: %d taps", taps);
+#define CR_LAUNCH(TAPS)                                                                                                                                     \
+    do {                                                                                                                                                    \
+        if (vec) ti_launch(conv_rows_kernel<T, 4, TAPS>, grid, dim3(threads), 0, stream, (T*)out, (const T*)h, (const T*)conv, taps, hist, hist_stride, cu_seqlens, seq_slots, B, n, size); \
+        else ti_launch(conv_rows_kernel<T, 1, TAPS>, grid, dim3(threads), 0, stream, (T*)out, (const T*)h, (const T*)conv, taps, hist, hist_stride, cu_seqlens, seq_slots, B, n, size); \
+    } while (0)
     TI_DISPATCH_DTYPE(dtype, {
         const uintptr_t mask = sizeof(T) == 2 ? 7 : 15;
         const bool vec = size % 4 == 0 && (((uintptr_t)out | (uintptr_t)h | (uintptr_t)conv) & mask) == 0 && aligned16(hist) && hist_stride % 4 == 0;
         const int per = vec ? 4 : 1, threads = 128;
-        const dim3 grid((size / per + threads - 1) / threads + (size % per ? 1 : 0), (n + CR_TOKENS - 1) / CR_TOKENS);
-        if (vec) ti_launch(conv_rows_kernel<T, 4>, grid, dim3(threads), 0, stream, (T*)out, (const T*)h, (const T*)conv, taps, hist, hist_stride, cu_seqlens, seq_slots, B, n, size);
-        else ti_launch(conv_rows_kernel<T, 1>, grid, dim3(threads), 0, stream, (T*)out, (const T*)h, (const T*)conv, taps, hist, hist_stride, cu_seqlens, seq_slots, B, n, size);
+        const dim3 grid((size / per + threads - 1) / threads, (n + CR_TOKENS - 1) / CR_TOKENS);
+        switch (taps) {
+            case 1: CR_LAUNCH(1); break;
+            case 2: CR_LAUNCH(2); break;
+            case 3: CR_LAUNCH(3); break;
+            case 4: CR_LAUNCH(4); break;
+            default: CR_LAUNCH(0); break;
+        }
     });
+#undef CR_LAUNCH
     return ti_check_launch("conv_rows");
 }
