@@ -19,12 +19,13 @@
 // q and k are rotated by the token's position and scaled while they are staged, in 32-bit. L is summed in 64-bit: a difference of two
 // large sums must not lose the small decay between neighbours.
 #include "common.cuh"
+#include "mma_util.cuh"
 
 #define MC_TOKENS 64
 #define MC_SLAB 128              // key rows and value columns staged at once
 #define MC_PITCH (MC_SLAB + 4)   // floats between staged rows: eight rows' 16-byte pieces lie in different banks
 #define MC_THREADS 256
-#define MC_S_ROWS 32             // rows of the state staged at once
+#define MC_S_ROWS 16             // rows of the state staged at once, twice: one piece is on its way while the other is worked on
 #define MC_FLOOR 1e-6f
 
 struct ChunkArgs {
@@ -108,6 +109,7 @@ __device__ __forceinline__ void stage_qk(const ChunkArgs& a, float* dst, int off
     if constexpr (VECTORS) {
         constexpr int VEC = Vec16<T>::N;
         const int per = width / VEC;
+#pragma unroll 4
         for (int e = threadIdx.x; e < MC_TOKENS * per; e += MC_THREADS) {
             const int s = e / per, d = d0 + (e % per) * VEC;
             float* out = dst + s * MC_PITCH + d - d0;
@@ -160,6 +162,7 @@ template <typename T, bool VECTORS>
 __device__ __forceinline__ void stage_v(const ChunkArgs& a, float* dst, const float* weight, int h, int t0, int count, int v0) {
     constexpr int VEC = VECTORS ? Vec16<T>::N : 1;
     const int per = MC_SLAB / VEC;
+#pragma unroll 4
     for (int e = threadIdx.x; e < MC_TOKENS * per; e += MC_THREADS) {
         const int s = e / per, c = (e % per) * VEC;
         float* out = dst + s * MC_SLAB + c;
@@ -301,7 +304,7 @@ template <typename T, bool VECTORS>
 __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(ChunkArgs a, ChunkOut out) {
     extern __shared__ __align__(16) float smem[];
     float* qs = smem;                                    // [64][MC_PITCH]
-    float* ks = qs + MC_TOKENS * MC_PITCH;               // [64][MC_PITCH]; later P [64][68] and a piece of the state [32][MC_SLAB]
+    float* ks = qs + MC_TOKENS * MC_PITCH;               // [64][MC_PITCH]; later P [64][68] and two pieces of the state [MC_S_ROWS][MC_SLAB]
     float* vs = ks + MC_TOKENS * MC_PITCH;               // [64][MC_SLAB]
     float* P = ks;
     float* ss = ks + MC_TOKENS * (MC_TOKENS + 4);
@@ -356,6 +359,25 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(Chu
         }
     }
     __syncthreads();                                     // the staged keys are done with: P and the state's pieces take their place
+    const int pieces = (D + MC_S_ROWS - 1) / MC_S_ROWS;
+    auto fetch = [&](int piece) {                        // rows piece * MC_S_ROWS .. of the state, zeros beyond
+        float* dst = ss + (piece & 1) * MC_S_ROWS * MC_SLAB;
+        const int d = piece * MC_S_ROWS;
+        if (V % 4 == 0) {
+            for (int e = threadIdx.x; e < MC_S_ROWS * (MC_SLAB / 4); e += MC_THREADS) {
+                const int r = e / (MC_SLAB / 4), c = (e % (MC_SLAB / 4)) * 4;
+                if (d + r < D && v0 + c < V) cp_async16(smem_u32(dst + r * MC_SLAB + c), state + (size_t)(d + r) * V + v0 + c);
+                else *reinterpret_cast<float4*>(dst + r * MC_SLAB + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        } else {
+            for (int e = threadIdx.x; e < MC_S_ROWS * MC_SLAB; e += MC_THREADS) {
+                const int r = e / MC_SLAB, c = e % MC_SLAB;
+                dst[e] = d + r < D && v0 + c < V ? __ldcg(state + (size_t)(d + r) * V + v0 + c) : 0.f;
+            }
+        }
+        cp_async_commit();
+    };
+    fetch(0);
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -369,45 +391,31 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(Chu
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
-    for (int d0 = 0; d0 < D; d0 += MC_SLAB) {
-        if (D > MC_SLAB) {                               // (with one slab q is still staged)
+    for (int piece = 0; piece < pieces; ++piece) {
+        const int d = piece * MC_S_ROWS, in_slab = d % MC_SLAB;
+        cp_async_wait<0>();
+        __syncthreads();                                 // this piece is there, and everyone is done with the one before
+        if (piece + 1 < pieces) fetch(piece + 1);
+        if (D > MC_SLAB && in_slab == 0) {               // (with one slab q is still staged)
+            stage_qk<T, VECTORS>(a, qs, a.q_off, a.q_scale, h, t0, count, d);
             __syncthreads();
-            stage_qk<T, VECTORS>(a, qs, a.q_off, a.q_scale, h, t0, count, d0);
         }
-        const int slab = min(MC_SLAB, D - d0);
-        for (int r0 = 0; r0 < slab; r0 += MC_S_ROWS) {
-            __syncthreads();
-            const int rows = min(MC_S_ROWS, slab - r0);
-            if (V % 4 == 0) {
-                for (int e = threadIdx.x; e < MC_S_ROWS * (MC_SLAB / 4); e += MC_THREADS) {
-                    const int r = e / (MC_SLAB / 4), c = (e % (MC_SLAB / 4)) * 4;
-                    float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (r < rows && v0 + c < V) t = __ldcg(reinterpret_cast<const float4*>(state + (size_t)(d0 + r0 + r) * V + v0 + c));
-                    *reinterpret_cast<float4*>(ss + r * MC_SLAB + c) = t;
-                }
-            } else {
-                for (int e = threadIdx.x; e < MC_S_ROWS * MC_SLAB; e += MC_THREADS) {
-                    const int r = e / MC_SLAB, c = e % MC_SLAB;
-                    ss[e] = r < rows && v0 + c < V ? __ldcg(state + (size_t)(d0 + r0 + r) * V + v0 + c) : 0.f;
-                }
-            }
-            __syncthreads();
-            const int padded = (rows + 3) / 4 * 4;       // (the staged q is zero beyond the head)
+        const float* sp = ss + (piece & 1) * MC_S_ROWS * MC_SLAB;
+        const int padded = min(MC_S_ROWS, (D - d + 3) / 4 * 4);          // (the staged q is zero beyond the head)
 #pragma unroll 2
-            for (int r = 0; r < padded; r += 4) {
-                float4 q4[4];
+        for (int r = 0; r < padded; r += 4) {
+            float4 q4[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) q4[i] = *reinterpret_cast<const float4*>(qs + (ry * 4 + i) * MC_PITCH + r0 + r);
+            for (int i = 0; i < 4; ++i) q4[i] = *reinterpret_cast<const float4*>(qs + (ry * 4 + i) * MC_PITCH + in_slab + r);
 #pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    const float4 s0 = *reinterpret_cast<const float4*>(ss + (r + k) * MC_SLAB + cx * 4), s1 = *reinterpret_cast<const float4*>(ss + (r + k) * MC_SLAB + 64 + cx * 4);
-                    const float sv[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
+            for (int k = 0; k < 4; ++k) {
+                const float4 s0 = *reinterpret_cast<const float4*>(sp + (r + k) * MC_SLAB + cx * 4), s1 = *reinterpret_cast<const float4*>(sp + (r + k) * MC_SLAB + 64 + cx * 4);
+                const float sv[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const float q = k == 0 ? q4[i].x : k == 1 ? q4[i].y : k == 2 ? q4[i].z : q4[i].w;
+                for (int i = 0; i < 4; ++i) {
+                    const float q = k == 0 ? q4[i].x : k == 1 ? q4[i].y : k == 2 ? q4[i].z : q4[i].w;
 #pragma unroll
-                        for (int j = 0; j < 8; ++j) acc[i][j] = fmaf(q, sv[j], acc[i][j]);
-                    }
+                    for (int j = 0; j < 8; ++j) acc[i][j] = fmaf(q, sv[j], acc[i][j]);
                 }
             }
         }
