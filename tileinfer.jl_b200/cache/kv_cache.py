@@ -18,6 +18,9 @@ keys). Its pool is therefore sized for ``max_seqs`` windows plus the tokens of o
 for ``max_tokens``; a long step is held chunk by chunk (``reserve`` checks the peak over the
 chunks, ``prepare`` takes each chunk's pages).
 
+A window may come with ``keep_first`` positions at a sequence's start that every query goes on seeing: their
+pages (in whole release units) are held until the sequence ends.
+
 The reference has one group, one sequence per step and a block table per ``Sequence``
 object (src/kv/block_manager.jl:13-16); slots, groups and the per-sequence state are this
 library's own.
@@ -107,6 +110,12 @@ class _Pages:
         return bool(self._g._api.group_page_is_held(self._g._book, self._g.book_index, page))
 
 
+def kept_pages(request: CacheRequest, cache) -> int:
+    """Pages at a sequence's start that stay visible beside the window, in whole release units."""
+    unit = cache.page_size * cache.release_granule
+    return -(-request.keep_first // unit) * cache.release_granule if request.window else 0
+
+
 @register_cache_kind("paged_kv")
 class PagedGroup:
     paged, rolls_back = True, True
@@ -116,12 +125,12 @@ class PagedGroup:
         pages = cache.num_pages
         if request.window and cache.max_step_tokens:
             # Each sequence: the pages that its window touches, the release unit's slack and the
-            # page that it writes to; plus the tokens of one step.
-            per_seq = -(-(request.window - 1) // cache.page_size) + cache.release_granule + 1
+            # page that it writes to, and the kept pages at its start; plus the tokens of one step.
+            per_seq = -(-(request.window - 1) // cache.page_size) + cache.release_granule + 1 + kept_pages(request, cache)
             pages = min(pages, cache.max_seqs * per_seq + -(-cache.max_step_tokens // cache.page_size))
         max_pages_per_seq = -(-cache.max_seq_len // cache.page_size)
-        bi = cache._api.cache_add_group(cache._book, pages, cache.page_size, request.window or 0, cache.release_granule,
-                                        max_pages_per_seq)
+        bi = cache._api.cache_add_group(cache._book, pages, cache.page_size, request.window or 0,
+                                        request.keep_first if request.window else 0, cache.release_granule, max_pages_per_seq)
         return cls(index, cache._book, bi, request, layers, pages, cache.page_size, cache.max_seqs, max_pages_per_seq,
                    cache.dtype, cache.device, cache.release_granule)
 
@@ -172,12 +181,12 @@ class PagedGroup:
 
     @property
     def first(self) -> Dict[int, int]:
-        """Logical index of each sequence's first page that is still held (sequences that gave pages back only)."""
+        """Logical index of each sequence's first page that is still held behind the kept ones (sequences that gave pages back only)."""
         firsts = {s: self._api.group_first(self._book, self.book_index, s) for s in range(self.max_seqs)}
         return {s: f for s, f in firsts.items() if f}
 
     def first_needed_page(self, length: int) -> int:
-        """Logical index of the first page that a query at position ``length`` or later can read."""
+        """Logical index of the first page that a query at position ``length`` or later can read (kept pages aside)."""
         if not self.window:
             return 0
         key = max(0, length - self.window + 1)

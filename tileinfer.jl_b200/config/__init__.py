@@ -3,6 +3,7 @@ from .registry import (Architecture, config_from_dict, load_config, register_arc
                        registered_architectures, resolve_architecture)
 from .fasodra import FasodraConfig
 from .midisun import MidisunConfig
+from .pemarax import PemaraxConfig
 from .sozanex import SozanexConfig
 from .spec import (FeedForwardSpec, LayerSpec, Llama3RopeScaling, MixerSpec, ModelSpec, NormSpec, PassInputSpec, PositionSpec,
                    TensorDecl, TokenInputSpec, YarnRopeScaling)

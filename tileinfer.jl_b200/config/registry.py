@@ -15,6 +15,7 @@ from typing import Any, Callable, Dict, Mapping, Optional
 from .apertus import ApertusConfig, ConfigError
 from .fasodra import FasodraConfig
 from .midisun import MidisunConfig
+from .pemarax import PemaraxConfig
 from .vogilix import VogilixConfig
 from .sozanex import SozanexConfig
 from .zudepel import ZudepelConfig
@@ -79,3 +80,4 @@ register_architecture(ZudepelConfig.architecture, ZudepelConfig, model_type=Zude
 register_architecture(SozanexConfig.architecture, SozanexConfig, model_type=SozanexConfig.model_type)
 register_architecture(FasodraConfig.architecture, FasodraConfig, model_type=FasodraConfig.model_type)
 register_architecture(MidisunConfig.architecture, MidisunConfig, model_type=MidisunConfig.model_type)
+register_architecture(PemaraxConfig.architecture, PemaraxConfig, model_type=PemaraxConfig.model_type)

@@ -71,20 +71,21 @@ __global__ void __launch_bounds__(AD_THREADS) attention_decode_kernel(
     int first_key = (window > 0 && kv_len > window) ? kv_len - window : 0;
     if (ex.chunk > 0 && kv_len > 0) first_key = max(first_key, ((kv_len - 1) / ex.chunk) * ex.chunk);       // the chunk of the step's token
     const int t_begin = first_key / AD_PAGE, t_end = (kv_len + AD_PAGE - 1) / AD_PAGE;
-    const int n_tiles = t_end - t_begin;
-    const int my_lo = t_begin + (int)((long long)n_tiles * split / parts);
-    const int my_hi = t_begin + (int)((long long)n_tiles * (split + 1) / parts);
+    // The pages to walk: those of the kept first keys that lie before the window's, then [t_begin, t_end).
+    const int kept = min((ex.keep + AD_PAGE - 1) / AD_PAGE, t_begin), n_tiles = kept + t_end - t_begin;
+    const int my_lo = (int)((long long)n_tiles * split / parts), my_hi = (int)((long long)n_tiles * (split + 1) / parts);
+    auto tile_at = [&](int i) { return i < kept ? i : t_begin + i - kept; };
     const int* table = block_table + (size_t)__ldcg(seq_slots + b) * table_stride;
     bool waited = false;
 
-    auto issue = [&](int tile, int stage) {
-        if (tile < my_hi) {
-            if (tile == t_end - 1 && !waited) {              // the page that this step writes to
+    auto issue = [&](int i, int stage) {
+        if (i < my_hi) {
+            if (i == n_tiles - 1 && !waited) {              // the page that this step writes to
                 pdl_wait();
                 pdl_launch_dependents();
                 waited = true;
             }
-            const size_t base = ((size_t)__ldcg(table + tile) * nkv + kvh) * AD_PAGE * D;
+            const size_t base = ((size_t)__ldcg(table + tile_at(i)) * nkv + kvh) * AD_PAGE * D;
             load_tile<D>(tiles + (size_t)stage * 2 * SM::TILE, k_cache + base);
             load_tile<D>(tiles + (size_t)stage * 2 * SM::TILE + SM::TILE, v_cache + base);
         }
@@ -124,12 +125,12 @@ __global__ void __launch_bounds__(AD_THREADS) attention_decode_kernel(
     const float slope0 = ex.slope != nullptr ? ex.slope[head0 + (g < group ? g : 0)] : 0.f;
     const float slope1 = ex.slope != nullptr ? ex.slope[head0 + (g + 8 < group ? g + 8 : 0)] : 0.f;
 
-    for (int tile = my_lo; tile < my_hi; ++tile) {
-        const int stage = (tile - my_lo) % SM::STAGES;
+    for (int step = my_lo; step < my_hi; ++step) {
+        const int stage = (step - my_lo) % SM::STAGES, tile = tile_at(step);
         cp_async_wait<SM::STAGES - 2>();
         __syncthreads();
         // The stage freed by the previous iteration is refilled while this one is used.
-        issue(tile + SM::STAGES - 1, (tile - my_lo + SM::STAGES - 1) % SM::STAGES);
+        issue(step + SM::STAGES - 1, (step - my_lo + SM::STAGES - 1) % SM::STAGES);
         const bf16* kt = tiles + (size_t)stage * 2 * SM::TILE;
         const bf16* vt = kt + SM::TILE;
 
@@ -279,14 +280,16 @@ static int launch_decode(bf16* out, const bf16* q, const bf16* k, const bf16* v,
 // pairs; seq_work[sequence] = first slot << 8 | parts; a sequence's slots are consecutive. Without them every sequence takes `splits` equal parts.
 // `sink` [nq] float (or null): one more term exp(sink[head]) in every softmax's denominator, with no key and no value.
 // `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`, `cap`, `slope` [nq] (times log2 e): see AttnExtras.
-extern "C" int ti_attention_decode_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+// `keep`: beside a window, the first `keep` positions stay visible.
+extern "C" int ti_attention_decode_kept(void* out, const void* q, const void* k_cache, const void* v_cache,
                                           const int* block_table, int table_stride, const int* seq_slots, const int* kv_lens,
                                           const int* work, const int* seq_work, float* ws_o, float* ws_ml, float scale, int B,
                                           int nq, int nkv, int D, int page_size, int splits, int window, const float* sink, int chunk,
-                                          const float* dist_bias, int bias_len, float cap, const float* slope, cudaStream_t stream) {
+                                          const float* dist_bias, int bias_len, float cap, const float* slope, int keep, cudaStream_t stream) {
     if (B == 0) return 0;
+    TI_REQUIRE(keep >= 0 && (keep == 0 || chunk == 0), "attention_decode: kept positions beside a window, not beside chunks");
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention_decode: chunk %d, bias table of %d", chunk, bias_len);
-    const AttnExtras ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope);
+    const AttnExtras ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope, window > 0 ? keep : 0);
     if (page_size != AD_PAGE || nq % nkv != 0 || nq / nkv > 128 || D % 16 != 0 || B > 32767 || (long long)nkv * ((nq / nkv + 15) / 16) > 65535) {
         ti_fail("attention_decode takes page size %d, at most 128 query heads per KV head and head sizes in steps of 16; "
                 "got page %d, %d/%d heads, head size %d", AD_PAGE, page_size, nq, nkv, D);
@@ -307,6 +310,15 @@ extern "C" int ti_attention_decode_ruled(void* out, const void* q, const void* k
             return 2;
     }
 #undef AD_CASE
+}
+
+extern "C" int ti_attention_decode_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                         const int* block_table, int table_stride, const int* seq_slots, const int* kv_lens,
+                                         const int* work, const int* seq_work, float* ws_o, float* ws_ml, float scale, int B,
+                                         int nq, int nkv, int D, int page_size, int splits, int window, const float* sink, int chunk,
+                                         const float* dist_bias, int bias_len, float cap, const float* slope, cudaStream_t stream) {
+    return ti_attention_decode_kept(out, q, k_cache, v_cache, block_table, table_stride, seq_slots, kv_lens, work, seq_work, ws_o, ws_ml, scale,
+                                    B, nq, nkv, D, page_size, splits, window, sink, chunk, dist_bias, bias_len, cap, slope, 0, stream);
 }
 
 extern "C" int ti_attention_decode_biased(void* out, const void* q, const void* k_cache, const void* v_cache,

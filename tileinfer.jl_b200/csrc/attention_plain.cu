@@ -30,7 +30,7 @@ __global__ void attention_plain_kernel(T* __restrict__ out, const T* q, const T*
                                        const int* positions, float scale, int nq, int nkv, int D,
                                        int page_size, int window, const float* __restrict__ sink, int chunk,
                                        const float* __restrict__ dist_bias, int bias_len, float cap,
-                                       const float* __restrict__ slope) {
+                                       const float* __restrict__ slope, int keep) {
     extern __shared__ float smem[];
     float* qs = smem;                          // [AP_HEADS][D]
     float* sc = smem + AP_HEADS * D;           // [AP_HEADS][AP_CHUNK]
@@ -60,10 +60,12 @@ __global__ void attention_plain_kernel(T* __restrict__ out, const T* q, const T*
     // Chunked visibility: only the keys of the query's own chunk of `chunk` positions, counted from the sequence's start.
     if (chunk > 0) first = max(first, (p / chunk) * chunk);
     const bool wide = D % Vec16<T>::N == 0 && (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0;
-    // Chunk borders are multiples of AP_CHUNK in absolute positions.
-    for (int c0 = (first / AP_CHUNK) * AP_CHUNK; c0 <= p; c0 += AP_CHUNK) {
-        const int lo = c0 > first ? c0 : first;
-        const int hi = (c0 + AP_CHUNK - 1 < p) ? c0 + AP_CHUNK - 1 : p;       // inclusive
+    // Chunk borders are multiples of AP_CHUNK in absolute positions. The kept first keys that lie before the window's come first.
+    const int kept = min(keep, first);
+    for (int part = kept > 0 ? 0 : 1; part < 2; ++part)
+    for (int begin = part == 0 ? 0 : first, end = part == 0 ? kept - 1 : p, c0 = (begin / AP_CHUNK) * AP_CHUNK; c0 <= end; c0 += AP_CHUNK) {
+        const int lo = c0 > begin ? c0 : begin;
+        const int hi = (c0 + AP_CHUNK - 1 < end) ? c0 + AP_CHUNK - 1 : end;       // inclusive
         float cmax[AP_HEADS];
 #pragma unroll
         for (int h = 0; h < AP_HEADS; ++h) cmax[h] = -INFINITY;
@@ -158,13 +160,15 @@ __global__ void attention_plain_kernel(T* __restrict__ out, const T* q, const T*
 // `chunk` > 0: a key is visible only inside the query's chunk of so many positions; `dist_bias` [nq][bias_len] float: added to
 // the scaled score by the distance between query and key (null: none). `cap` > 0: the scaled score s becomes cap tanh(s / cap) before
 // any bias; `slope` [nq] float (null: none): slope[head] * distance is taken off after the cap.
-extern "C" int ti_attention_plain_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+// `keep`: beside a window, the first `keep` positions stay visible.
+extern "C" int ti_attention_plain_kept(void* out, const void* q, const void* k_cache, const void* v_cache,
                                         const int* block_table, int table_stride, const int* tok_slot, const int* positions,
                                          float scale, int n_tokens, int nq, int nkv, int D, int page_size, int window,
                                          const float* sink, int chunk, const float* dist_bias, int bias_len, float cap, const float* slope,
-                                        int dtype, cudaStream_t stream) {
+                                        int keep, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention: chunk %d, bias table of %d", chunk, bias_len);
+    TI_REQUIRE(keep >= 0 && (keep == 0 || chunk == 0), "attention: kept positions beside a window, not beside chunks");
     TI_REQUIRE(D > 0 && D <= AP_MAX_D, "attention: head_dim %d exceeds %d", D, AP_MAX_D);
     TI_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention: %d query heads do not divide into %d KV heads", nq, nkv);
     const int sets = (nq / nkv + AP_HEADS - 1) / AP_HEADS;
@@ -173,8 +177,17 @@ extern "C" int ti_attention_plain_ruled(void* out, const void* q, const void* k_
     const size_t smem = (size_t)AP_HEADS * (D + AP_CHUNK) * sizeof(float);
     TI_DISPATCH_DTYPE(dtype, (ti_launch(attention_plain_kernel<T>, dim3(grid), dim3(AP_THREADS), smem, stream, 
                                  (T*)out, (const T*)q, (const T*)k_cache, (const T*)v_cache, block_table, table_stride,
-                                 tok_slot, positions, scale, nq, nkv, D, page_size, window, sink, chunk, dist_bias, bias_len, cap, slope)));
+                                 tok_slot, positions, scale, nq, nkv, D, page_size, window, sink, chunk, dist_bias, bias_len, cap, slope, window > 0 ? keep : 0)));
     return ti_check_launch("attention_plain");
+}
+
+extern "C" int ti_attention_plain_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                        const int* block_table, int table_stride, const int* tok_slot, const int* positions,
+                                        float scale, int n_tokens, int nq, int nkv, int D, int page_size, int window,
+                                        const float* sink, int chunk, const float* dist_bias, int bias_len, float cap, const float* slope,
+                                        int dtype, cudaStream_t stream) {
+    return ti_attention_plain_kept(out, q, k_cache, v_cache, block_table, table_stride, tok_slot, positions, scale, n_tokens, nq, nkv, D, page_size,
+                                   window, sink, chunk, dist_bias, bias_len, cap, slope, 0, dtype, stream);
 }
 
 extern "C" int ti_attention_plain_biased(void* out, const void* q, const void* k_cache, const void* v_cache,

@@ -114,23 +114,26 @@ __global__ void __launch_bounds__(PF_THREADS, 1) attention_prefill_kernel(
     const int pos_first = start + j0, pos_last = start + j0 + n_tok - 1;
     const int key_lo = first_seen(pos_first), key_lo_last = first_seen(pos_last);
     const int t_lo = key_lo / PF_PAGE, t_hi = pos_last / PF_PAGE + 1;
+    // The walk's pages: those of the kept first keys that lie before the window's, then [t_lo, t_hi).
+    const int kept = min((ex.keep + PF_PAGE - 1) / PF_PAGE, t_lo), steps = kept + t_hi - t_lo;
+    auto tile_at = [&](int i) { return i < kept ? i : t_lo + i - kept; };
 
-    auto issue = [&](int tile, int stage) {
-        if (tile < t_hi) {
-            const size_t base = ((size_t)__ldcg(table + tile) * nkv + kvh) * PF_PAGE * D;
+    auto issue = [&](int i, int stage) {
+        if (i < steps) {
+            const size_t base = ((size_t)__ldcg(table + tile_at(i)) * nkv + kvh) * PF_PAGE * D;
             pf_load_tile<D>(tiles + (size_t)stage * 2 * SM::TILE, k_cache + base);
             pf_load_tile<D>(tiles + (size_t)stage * 2 * SM::TILE + SM::TILE, v_cache + base);
         }
         cp_async_commit();
     };
 #pragma unroll
-    for (int s = 0; s < SM::STAGES - 1; ++s) issue(t_lo + s, s);
+    for (int s = 0; s < SM::STAGES - 1; ++s) issue(s, s);
 
-    for (int tile = t_lo; tile < t_hi; ++tile) {
-        const int stage = (tile - t_lo) % SM::STAGES;
+    for (int step = 0; step < steps; ++step) {
+        const int stage = step % SM::STAGES, tile = tile_at(step);
         cp_async_wait<SM::STAGES - 2>();
         __syncthreads();
-        issue(tile + SM::STAGES - 1, (tile - t_lo + SM::STAGES - 1) % SM::STAGES);
+        issue(step + SM::STAGES - 1, (step + SM::STAGES - 1) % SM::STAGES);
         const bf16* kt = tiles + (size_t)stage * 2 * SM::TILE;
         const bf16* vt = kt + SM::TILE;
 
@@ -174,8 +177,8 @@ __global__ void __launch_bounds__(PF_THREADS, 1) attention_prefill_kernel(
                     c += bias1[min(max(pos1 - key, 0), ex.bias_len - 1)];
                 }
                 if (need_mask) {
-                    if (key > pos0 || key < lo0) a = -INFINITY;
-                    if (key > pos1 || key < lo1) c = -INFINITY;
+                    if (key > pos0 || (key < lo0 && key >= ex.keep)) a = -INFINITY;
+                    if (key > pos1 || (key < lo1 && key >= ex.keep)) c = -INFINITY;
                 }
                 s[nt][j] = a; s[nt][2 + j] = c;
                 mx0 = fmaxf(mx0, a); mx1 = fmaxf(mx1, c);
@@ -259,13 +262,15 @@ static int launch_prefill(bf16* out, const bf16* q, const bf16* k, const bf16* v
 // kernel takes (the caller then runs the plain kernel).
 // `sink` [nq] float (or null): one more term exp(sink[head]) in every softmax's denominator.
 // `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`, `cap`, `slope` [nq] (times log2 e): see AttnExtras.
-extern "C" int ti_attention_prefill_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+// `keep`: beside a window, the first `keep` positions stay visible.
+extern "C" int ti_attention_prefill_kept(void* out, const void* q, const void* k_cache, const void* v_cache,
                                          const int* block_table, int table_stride, const int* seq_slots,
                                          const int* cu_seqlens, const int* kv_lens, int n_seqs, int total_tiles, float scale,
                                          int nq, int nkv, int D, int page_size, int window, const float* sink, int chunk, const float* dist_bias, int bias_len,
-                                         float cap, const float* slope, cudaStream_t stream) {
-    const AttnExtras ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope);
+                                         float cap, const float* slope, int keep, cudaStream_t stream) {
+    const AttnExtras ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope, window > 0 ? keep : 0);
     if (n_seqs == 0 || total_tiles == 0) return 0;
+    TI_REQUIRE(keep >= 0 && (keep == 0 || chunk == 0), "attention_prefill: kept positions beside a window, not beside chunks");
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention_prefill: chunk %d, bias table of %d", chunk, bias_len);
     if (page_size != PF_PAGE || nq % nkv != 0 || nq / nkv > PF_ROWS || D % 16 != 0 || nkv > 65535) {
         ti_fail("attention_prefill takes page size %d, at most %d query heads per KV head and head sizes in steps of 16; "
@@ -285,6 +290,15 @@ extern "C" int ti_attention_prefill_ruled(void* out, const void* q, const void* 
             return 2;
     }
 #undef PF_CASE
+}
+
+extern "C" int ti_attention_prefill_ruled(void* out, const void* q, const void* k_cache, const void* v_cache,
+                                          const int* block_table, int table_stride, const int* seq_slots,
+                                          const int* cu_seqlens, const int* kv_lens, int n_seqs, int total_tiles, float scale,
+                                          int nq, int nkv, int D, int page_size, int window, const float* sink, int chunk, const float* dist_bias,
+                                          int bias_len, float cap, const float* slope, cudaStream_t stream) {
+    return ti_attention_prefill_kept(out, q, k_cache, v_cache, block_table, table_stride, seq_slots, cu_seqlens, kv_lens, n_seqs, total_tiles,
+                                     scale, nq, nkv, D, page_size, window, sink, chunk, dist_bias, bias_len, cap, slope, 0, stream);
 }
 
 extern "C" int ti_attention_prefill_biased(void* out, const void* q, const void* k_cache, const void* v_cache,

@@ -166,11 +166,16 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
     int key_lo = p.window > 0 ? max(0, start + t0 - p.window + 1) : 0;
     if (p.ex.chunk > 0) key_lo = max(key_lo, ((start + t0) / p.ex.chunk) * p.ex.chunk);        // the chunk of the block's first token
     const int j_lo = key_lo / KEYS, j_hi = (key_hi + KEYS - 1) / KEYS;
+    // The steps of the walk, numbered j_first .. j_hi - 1: the tiles of the kept first keys that lie before the window's, then [j_lo, j_hi).
+    const int j_first = j_lo - min((p.ex.keep + KEYS - 1) / KEYS, j_lo);
     const int n_pages = (kv_len + PAGE - 1) / PAGE;
     // With a slope by distance the nearest keys come first: a row's largest scores are then among the first it meets, and its output does
     // not have to be rescaled from tile to tile.
     const bool backward = p.ex.slope != nullptr;
-    auto tile_of = [&](int j) { return backward ? j_hi - 1 - (j - j_lo) : j; };
+    auto tile_of = [&](int j) {
+        const int u = backward ? j_hi - 1 - (j - j_first) : j;
+        return u < j_lo ? u - j_first : u;
+    };
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -208,10 +213,10 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
             // what stands in shared memory must be finite.
             const int* table = p.table + (long long)slot * p.table_stride;
             int page[KEYS / PAGE], next_page[KEYS / PAGE];
-            for (int pg = 0; pg < KEYS / PAGE; ++pg) page[pg] = __ldcg(table + min(tile_of(j_lo) * (KEYS / PAGE) + pg, n_pages - 1));
+            for (int pg = 0; pg < KEYS / PAGE; ++pg) page[pg] = __ldcg(table + min(tile_of(j_first) * (KEYS / PAGE) + pg, n_pages - 1));
             bool ok = true;
-            int fill = 0;                                       // K_j is fill 2(j - j_lo), V_j the next one
-            for (int j = j_lo; ok && j < j_hi; ++j) {
+            int fill = 0;                                       // K_j is fill 2(j - j_first), V_j the next one
+            for (int j = j_first; ok && j < j_hi; ++j) {
                 // The next step's page numbers are on their way while this step's tiles are waited for.
                 for (int pg = 0; pg < KEYS / PAGE; ++pg)
                     next_page[pg] = j + 1 < j_hi ? __ldcg(table + min(tile_of(j + 1) * (KEYS / PAGE) + pg, n_pages - 1)) : 0;
@@ -249,7 +254,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
                 umma_commit(s_full0 + 8 * x);
             };
             bool ok = mbar_wait(q_full, 0, p.status, 2);
-            if (ok && j_lo < j_hi) {
+            if (ok && j_first < j_hi) {
                 ok = mbar_wait(kv_full0, 0, p.status, 3);
                 tc_fence_after();
                 if (ok) {
@@ -259,10 +264,10 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
                 }
             }
             int fill = 0;
-            for (int j = j_lo; ok && j < j_hi; ++j, fill += 2) {
+            for (int j = j_first; ok && j < j_hi; ++j, fill += 2) {
                 const int vbuf = (fill + 1) % RING, knext = (fill + 2) % RING;
                 const unsigned vphase = (unsigned)((fill + 1) / RING) & 1u, kphase = (unsigned)((fill + 2) / RING) & 1u;
-                const unsigned jphase = (unsigned)(j - j_lo) & 1u;
+                const unsigned jphase = (unsigned)(j - j_first) & 1u;
                 ok = mbar_wait(kv_full0 + 8 * vbuf, vphase, p.status, 4);
                 if (ok && j + 1 < j_hi) ok = mbar_wait(kv_full0 + 8 * knext, kphase, p.status, 6);
                 if (!ok) break;
@@ -274,7 +279,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
 #pragma unroll
                     for (int s = 0; s < KEYS / 16; ++s)         // 16 keys = 16 rows of 128 bytes further on
                         umma_bf16_ts(tmem_base + C::O_COL + x * D, tmem_base + x * KEYS + s * 8,
-                                     smem_desc_mn_sw128(va + s * 2048, C::HALF_BYTES, 1024), IDESC_PV, (j > j_lo || s > 0) ? 1u : 0u);
+                                     smem_desc_mn_sw128(va + s * 2048, C::HALF_BYTES, 1024), IDESC_PV, (j > j_first || s > 0) ? 1u : 0u);
                     umma_commit(o_done0 + 8 * x);
                     if (j + 1 < j_hi) issue_qk(x, knext);
                 }
@@ -300,8 +305,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
         const float score_scale = shaped ? 1.0f : p.scale_log2;
         const float slope = p.ex.slope != nullptr ? __ldg(p.ex.slope + min(head, p.heads - 1)) : 0.f;
         bool ok = true;
-        for (int j = j_lo; ok && j < j_hi; ++j) {
-            const unsigned jphase = (unsigned)(j - j_lo) & 1u;
+        for (int j = j_first; ok && j < j_hi; ++j) {
+            const unsigned jphase = (unsigned)(j - j_first) & 1u;
             ok = __all_sync(0xffffffffu, mbar_wait(s_full0 + 8 * x, jphase, p.status, 7));
             if (!ok) break;
             tc_fence_after();
@@ -353,7 +358,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         const int key = key0 + c * 32 + i;
-                        if (!(key <= k_hi && key >= k_lo)) r[c][i] = 0xff800000u;       // -inf: its weight is exactly zero
+                        if (!(key <= k_hi && (key >= k_lo || key < p.ex.keep))) r[c][i] = 0xff800000u;       // -inf: its weight is exactly zero
                     }
             }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // independent chains
@@ -363,7 +368,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
                 for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(r[c][i]));
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
             const float mt = fmaxf(fmaf(mx, score_scale, row_base), -1e30f);
-            if (j == j_lo) {
+            if (j == j_first) {
                 m_used = mt;
             } else if (__any_sync(0xffffffffu, mt > m_used + RESCALE_STEP)) {
                 // O must be complete (the previous step's second product) before it is rescaled.
@@ -414,8 +419,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_tc_kernel(const 
             __syncwarp();
             if (lane == 0) mbar_arrive(p_ready0 + 8 * x);
         }
-        if (ok && j_lo < j_hi) {
-            ok = __all_sync(0xffffffffu, mbar_wait(o_done0 + 8 * x, (unsigned)(j_hi - 1 - j_lo) & 1u, p.status, 9));
+        if (ok && j_first < j_hi) {
+            ok = __all_sync(0xffffffffu, mbar_wait(o_done0 + 8 * x, (unsigned)(j_hi - 1 - j_first) & 1u, p.status, 9));
             tc_fence_after();
         }
         if (ok) {
@@ -474,12 +479,14 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 // takes (head size 64 or 128, 1 to 128 query heads per KV head, pages of 64): the caller then runs the
 // kernel for all sizes.
 // `chunk`, `dist_bias` [nq][bias_len] (times log2 e), `bias_len`, `cap`, `slope` [nq] (times log2 e): see AttnExtras.
-extern "C" int ti_attention_prefill_tc_ruled(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,
+// `keep`: beside a window, the first `keep` positions stay visible.
+extern "C" int ti_attention_prefill_tc_kept(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,
                                               const int* block_table, int table_stride, const int* seq_slots,
                                               const int* cu_seqlens, const int* kv_lens, int n_seqs, int n_tokens, int total_blocks,
                                               float scale, int nq, int nkv, int D, int page_size, int window, int* status,
                                               const float* sink, int chunk, const float* dist_bias, int bias_len, float cap, const float* slope,
-                                             cudaStream_t stream) {
+                                             int keep, cudaStream_t stream) {
+    TI_REQUIRE(keep >= 0 && (keep == 0 || chunk == 0), "attention_prefill_tc: kept positions beside a window, not beside chunks");
     if (n_seqs == 0 || total_blocks == 0) return 0;
     TI_REQUIRE(chunk >= 0 && (dist_bias == nullptr || bias_len > 0), "attention_prefill_tc: chunk %d, bias table of %d", chunk, bias_len);
     const int group = nkv > 0 ? nq / nkv : 0;
@@ -494,7 +501,7 @@ extern "C" int ti_attention_prefill_tc_ruled(void* out, const void* q, const voi
     p.out = (bf16*)out; p.table = block_table; p.table_stride = table_stride; p.slots = seq_slots; p.cu_seqlens = cu_seqlens;
     p.kv_lens = kv_lens; p.n_seqs = n_seqs; p.heads = nq; p.kv_heads = nkv; p.group = group; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.sink = sink;
-    p.ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope);
+    p.ex = attn_extras(chunk, dist_bias, bias_len, scale, cap, slope, window > 0 ? keep : 0);
     CUtensorMap mq, mk, mv;
     {
         const unsigned long long dims[3] = {(unsigned long long)D, (unsigned long long)nq, (unsigned long long)n_tokens};
@@ -511,6 +518,17 @@ extern "C" int ti_attention_prefill_tc_ruled(void* out, const void* q, const voi
     }
     return D == 64 ? launch<64>(mq, mk, mv, (const bf16*)q, p, total_blocks, stream)
                    : launch<128>(mq, mk, mv, (const bf16*)q, p, total_blocks, stream);
+}
+
+extern "C" int ti_attention_prefill_tc_ruled(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,
+                                             const int* block_table, int table_stride, const int* seq_slots,
+                                             const int* cu_seqlens, const int* kv_lens, int n_seqs, int n_tokens, int total_blocks,
+                                             float scale, int nq, int nkv, int D, int page_size, int window, int* status,
+                                             const float* sink, int chunk, const float* dist_bias, int bias_len, float cap, const float* slope,
+                                             cudaStream_t stream) {
+    return ti_attention_prefill_tc_kept(out, q, k_cache, v_cache, n_pages, block_table, table_stride, seq_slots, cu_seqlens, kv_lens, n_seqs,
+                                        n_tokens, total_blocks, scale, nq, nkv, D, page_size, window, status, sink, chunk, dist_bias, bias_len,
+                                        cap, slope, 0, stream);
 }
 
 extern "C" int ti_attention_prefill_tc_biased(void* out, const void* q, const void* k_cache, const void* v_cache, int n_pages,

@@ -218,7 +218,8 @@ __host__ __forceinline__ bool aligned16(const void* p) { return ((uintptr_t)p & 
 // (null: none): entry [head][min(i - j, bias_len - 1)] is added to the scaled score; the kernels that work in base 2 get the
 // table already times log2(e). cap_out > 0: the scaled score s becomes cap * tanh(s / cap), before any bias; slope [heads] (null:
 // none): slope[head] * (i - j) is taken off afterwards. The kernels that work in base 2 read cap_in = 2 scale log2(e) / cap (it
-// multiplies the unscaled score), cap_out = cap log2(e) and slopes times log2(e).
+// multiplies the unscaled score), cap_out = cap log2(e) and slopes times log2(e). keep > 0: beside a window, the sequence's first
+// `keep` positions stay visible to every later query.
 struct AttnExtras {
     int chunk;
     const float* bias;
@@ -227,12 +228,14 @@ struct AttnExtras {
     float cap_small = 0.f;               // scores (unscaled) up to which |scale * score / cap| <= 1/2
     float cap_ratio2 = 0.f;              // (scale / cap)^2
     const float* slope = nullptr;
+    int keep = 0;
 };
-inline AttnExtras attn_extras(int chunk, const float* bias, int bias_len, float scale, float cap, const float* slope) {
+inline AttnExtras attn_extras(int chunk, const float* bias, int bias_len, float scale, float cap, const float* slope, int keep = 0) {
     AttnExtras ex = {chunk, bias, bias_len};
     if (cap > 0.f) { ex.cap_in = 2.f * scale * 1.4426950408889634f / cap; ex.cap_out = cap * 1.4426950408889634f; }
     if (cap > 0.f && scale != 0.f) { ex.cap_small = 0.5f * cap / (scale < 0.f ? -scale : scale); ex.cap_ratio2 = (scale / cap) * (scale / cap); }
     ex.slope = slope;
+    ex.keep = keep;
     return ex;
 }
 // cap log2(e) tanh(scale * raw / cap) as cap_out (1 - 2 / (1 + 2^(cap_in raw))): its error is a rounding of cap_out, whatever the score.

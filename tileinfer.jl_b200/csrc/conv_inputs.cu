@@ -4,7 +4,8 @@
 //   y_t[c] = T( sum_j conv[c][j] * u_(t - taps + 1 + j)[c] )   zeros before the sequence's start
 //   q, k  <- y / rms(y over the WHOLE row of q, or of k) * w    (weights as long as the row; optional)
 //            or, with head_norm, every head by itself: y_h / rms(y_h) * w, one weight of the head's size for all heads
-//   q, k  <- rotation of the first `rotary` elements of every head by the position's angles (optional)
+//   q, k  <- rotation of the first `rotary` elements of every head by the position's angles (optional); with norm_last the rotation
+//            comes first and the heads' norms after it
 //   q -> q_out [n, heads, Dp]; k, v -> their place in the paged cache [pages][kv_heads][page][Dp]
 //
 // Dp >= the query/key size and the value size: rows are filled up with zeros, which changes neither a score nor an output.
@@ -33,7 +34,7 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
     const T* __restrict__ q_norm_w, const T* __restrict__ k_norm_w, float eps, const float* __restrict__ cos_sin, int rotary,
     T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* positions, const int* slot_map,
     const int* cu_seqlens, const int* seq_slots, const int* kv_lens, int B, int nq, int nkv, int D, int V, int Dp, int page_size,
-    int write_kv, int head_norm, int shared_kv) {
+    int write_kv, int head_norm, int shared_kv, int interleaved, int norm_last) {
     extern __shared__ float y[];                       // [channels]
     __shared__ float scratch[33];
     const int t = blockIdx.x;
@@ -93,6 +94,21 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         }
         __syncthreads();
     }
+    const int half = rotary >> 1;
+    const float* cs = cos_sin != nullptr ? cos_sin + (size_t)p * rotary : nullptr;       // [half][2] = (cos, sin)
+    if (norm_last && cs != nullptr) {
+        // The pairs of every query and key head in place, a thread per pair.
+        __syncthreads();
+        for (int e = threadIdx.x; e < (nq + (write_kv ? nkv : 0)) * half; e += CI_THREADS) {
+            const int i = e % half;
+            float* src = y + (size_t)(e / half) * D;
+            const int a = interleaved ? 2 * i : i, c = interleaved ? 2 * i + 1 : i + half;
+            const float u = src[a], v = src[c];
+            src[a] = u * cs[2 * i] - v * cs[2 * i + 1];
+            src[c] = v * cs[2 * i] + u * cs[2 * i + 1];
+        }
+        cs = nullptr;                          // done
+    }
     if (head_norm) {
         // A warp per head: the order of a head's sum depends on the head's size alone.
         __syncthreads();
@@ -118,8 +134,6 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         else if (k_norm_w != nullptr) y[c] = y[c] * invk * to_f32(k_norm_w[c - Cq]);
     }
     __syncthreads();
-    const int half = rotary >> 1;
-    const float* cs = cos_sin != nullptr ? cos_sin + (size_t)p * rotary : nullptr;       // [half][2] = (cos, sin)
     // Queries and keys: heads of Dp elements, the first D from y (rotated where the rotation reaches), zeros after.
     const int qk_heads = nq + (write_kv ? nkv : 0);
     for (int e = threadIdx.x; e < qk_heads * Dp; e += CI_THREADS) {
@@ -129,8 +143,8 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
             const float* src = y + (size_t)head * D;   // key heads follow the query heads in y
             v = src[d];
             if (cs != nullptr && d < rotary) {
-                const int i = d < half ? d : d - half;
-                const float other = d < half ? -src[d + half] : src[d - half];
+                const int i = interleaved ? d >> 1 : (d < half ? d : d - half);
+                const float other = interleaved ? ((d & 1) ? src[d - 1] : -src[d + 1]) : (d < half ? -src[d + half] : src[d - half]);
                 v = v * cs[2 * i] + other * cs[2 * i + 1];
             }
         }
@@ -146,19 +160,22 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
 
 // proj [n, ld] of T: the step's projected rows, queries (nq * D) then, with write_kv, keys (nkv * D) and values (nkv * V);
 // bias and conv [channels, taps] in the same channel order (null: none; taps 0: no convolution); state [slots, taps - 1, channels]
-// float; cos_sin [positions, rotary / 2, 2] float (null: no rotation; pairs i, i + rotary / 2). head_norm: the norm weights are
+// float; cos_sin [positions, rotary / 2, 2] float (null: no rotation; pairs i, i + rotary / 2, or
+// with `interleaved` 2i, 2i + 1). norm_last: rotation before the heads' norms (head_norm). head_norm: the norm weights are
 // [D] and every head is normed by itself. shared_kv: there are no value rows; a token's values are its keys' rows before norm and
 // rotation.
 extern "C" int ti_conv_attention_inputs(const void* proj, long long ld, const void* bias, const void* conv, int taps, const float* state,
                                         const void* q_norm_w, const void* k_norm_w, float eps, const float* cos_sin, int rotary, void* q_out,
                                         void* k_cache, void* v_cache, const int* positions, const int* slot_map, const int* cu_seqlens,
                                         const int* seq_slots, const int* kv_lens, int n, int B, int nq, int nkv, int D, int V, int Dp,
-                                        int page_size, int write_kv, int head_norm, int shared_kv, int dtype, cudaStream_t stream) {
+                                        int page_size, int write_kv, int head_norm, int shared_kv, int interleaved, int norm_last, int dtype,
+                                        cudaStream_t stream) {
     if (n == 0) return 0;
     TI_REQUIRE(taps >= 0 && taps <= CI_MAX_TAPS && (taps <= 1 || state != nullptr) && (taps == 0 || conv != nullptr), "conv_attention_inputs: %d taps", taps);
     TI_REQUIRE(D > 0 && V > 0 && Dp >= D && Dp >= V && nq > 0 && nkv > 0, "conv_attention_inputs: heads of %d / %d in rows of %d", D, V, Dp);
     TI_REQUIRE(cos_sin == nullptr || (rotary >= 2 && rotary % 2 == 0 && rotary <= D), "conv_attention_inputs: rotation over %d of %d", rotary, D);
     TI_REQUIRE(!shared_kv || V == D, "conv_attention_inputs: values that are the keys' projection have the keys' size (%d, not %d)", D, V);
+    TI_REQUIRE(!norm_last || head_norm, "conv_attention_inputs: a norm after the rotation is built for heads normed one by one");
     const int C = nq * D + (write_kv ? nkv * (shared_kv ? D : D + V) : 0);
     const size_t smem = (size_t)C * sizeof(float);
     TI_REQUIRE(smem <= 160 * 1024, "conv_attention_inputs: %d channels", C);
@@ -167,7 +184,7 @@ extern "C" int ti_conv_attention_inputs(const void* proj, long long ld, const vo
         if (smem > 48 * 1024) cudaFuncSetAttribute(conv_attention_inputs_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         ti_launch(conv_attention_inputs_kernel<T, TAPS>, dim3(n), dim3(CI_THREADS), smem, stream, (const T*)proj, ld, (const T*)bias, (const T*)conv,  \
                   taps, state, (const T*)q_norm_w, (const T*)k_norm_w, eps, cos_sin, rotary, (T*)q_out, (T*)k_cache, (T*)v_cache, positions,       \
-                  slot_map, cu_seqlens, seq_slots, kv_lens, B, nq, nkv, D, V, Dp, page_size, write_kv, head_norm, shared_kv);                          \
+                  slot_map, cu_seqlens, seq_slots, kv_lens, B, nq, nkv, D, V, Dp, page_size, write_kv, head_norm, shared_kv, interleaved, norm_last);   \
     } while (0)
     TI_DISPATCH_DTYPE(dtype, {
         switch (taps) {

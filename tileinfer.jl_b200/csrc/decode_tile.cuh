@@ -40,7 +40,7 @@ __device__ __forceinline__ void decode_tile(const bf16* kt, const bf16* vt, cons
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
             const int key = key0 + 8 * nt + j;
-            const bool ok = key < kv_len && key >= first_key;
+            const bool ok = key < kv_len && (key >= first_key || key < ex.keep);
             float add0 = 0.f, add1 = 0.f;
             if (bias0 != nullptr && ok) {                    // the bias of the distance from the step's token, per row's head
                 const int dist = min(kv_len - 1 - key, bias_len - 1);

@@ -1,8 +1,8 @@
 // A 32-bit residual stream whose sublayers are added through a learned gate, normed in groups, with a short causal convolution over
 // time ahead of a mixer.
 //
-//   gated_add_norm32   x += (d + bias) * sigmoid(g + gbias);  h = T(G(x) * w), G: the row in `groups` equal parts, each divided by
-//                      its own sqrt(mean(part^2) + eps);  for one-token steps also hc = T(h + conv(h)) from and to the sequences' history
+//   gated_add_norm32   x += mult * (d + bias) * sigmoid(g + gbias);  h = T(G(x) * w), G: the row in `groups` equal parts, each divided by
+//                      its own sqrt(mean(part^2) + eps) (`offset`: times 1 + w);  for one-token steps also hc = T(h + conv(h)) from and to the sequences' history
 //   conv_rows          hc = T(h + conv(h)), conv(h)_t = sum_j c[j] * h_(t - taps + 1 + j) per channel, over a step's rows (rows before the
 //                      step from the history; its update is history_update, a launch of its own, since these blocks read it)
 //
@@ -92,7 +92,7 @@ __device__ __forceinline__ void branch_piece(const BranchRows& b, int row, int s
 
 template <typename T, int VEC>
 __global__ void gated_add_norm32_kernel(float* x, BranchRows d, BranchRows g, T* h, const T* __restrict__ w, float eps, int groups, ConvStep cs,
-                                        int size, int has_branch, int has_gate) {
+                                        int size, int has_branch, int has_gate, float mult, int offset) {
     extern __shared__ __align__(16) float row_d[];       // [size] the stream's new row, then [groups] sums' reciprocals, then partial sums
     const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     float* xr = x + (size_t)row * size;
@@ -112,7 +112,7 @@ __global__ void gated_add_norm32_kernel(float* x, BranchRows d, BranchRows g, T*
                 for (int e = 0; e < VEC; ++e) dv[e] = dv[e] / (1.0f + expf(-gv[e]));
             }
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) v[e] += dv[e];
+            for (int e = 0; e < VEC; ++e) v[e] = fmaf(mult, dv[e], v[e]);
             Piece<float, VEC>::store(xr + i, v);
         }
         Piece<float, VEC>::store(row_d + i, v);
@@ -144,7 +144,7 @@ __global__ void gated_add_norm32_kernel(float* x, BranchRows d, BranchRows g, T*
         float v[VEC], wv[VEC];
         Piece<T, VEC>::load(w + i, wv);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) v[e] = rnd<T>(row_d[i + e] * inv[(i + e) / per] * wv[e]);
+        for (int e = 0; e < VEC; ++e) v[e] = rnd<T>(row_d[i + e] * inv[(i + e) / per] * (offset ? 1.0f + wv[e] : wv[e]));
         Piece<T, VEC>::store(h + (size_t)row * size + i, v);
         if (cs.conv == nullptr) continue;
         // One token per sequence: row r is sequence r's token. A thread owns its channels' history: it reads and moves it on.
@@ -176,7 +176,7 @@ static int row_vec_ok(const BranchRows& b, int elem) {
 // update alone. conv null: no convolution.
 extern "C" int ti_gated_add_norm32(float* x, const void* d, const float* d_partials, int d_n, long long d_stride, const int* index, const float* scores,
                                    int per_row, const void* d_bias, const void* g, const float* g_partials, int g_n, long long g_stride,
-                                   const void* g_bias, void* h, const void* w, float eps, int groups, const void* conv, int taps, float* hist,
+                                   const void* g_bias, float mult, void* h, const void* w, int offset, float eps, int groups, const void* conv, int taps, float* hist,
                                    long long hist_stride, const int* seq_slots, void* conv_out, int n_rows, int size, int dtype, cudaStream_t stream) {
     if (n_rows == 0) return 0;
     TI_REQUIRE(size > 0 && size <= 40000 && groups >= 1 && groups <= 4096 && size % groups == 0, "gated_add_norm32: rows of %d in %d groups", size, groups);
@@ -199,8 +199,8 @@ extern "C" int ti_gated_add_norm32(float* x, const void* d, const float* d_parti
             cudaFuncSetAttribute(gated_add_norm32_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             cudaFuncSetAttribute(gated_add_norm32_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         }
-        if (vec) ti_launch(gated_add_norm32_kernel<T, 4>, dim3(n_rows), dim3(threads), smem, stream, x, db, gb, (T*)h, (const T*)w, eps, groups, cs, size, has_branch, has_gate);
-        else ti_launch(gated_add_norm32_kernel<T, 1>, dim3(n_rows), dim3(threads), smem, stream, x, db, gb, (T*)h, (const T*)w, eps, groups, cs, size, has_branch, has_gate);
+        if (vec) ti_launch(gated_add_norm32_kernel<T, 4>, dim3(n_rows), dim3(threads), smem, stream, x, db, gb, (T*)h, (const T*)w, eps, groups, cs, size, has_branch, has_gate, mult, offset);
+        else ti_launch(gated_add_norm32_kernel<T, 1>, dim3(n_rows), dim3(threads), smem, stream, x, db, gb, (T*)h, (const T*)w, eps, groups, cs, size, has_branch, has_gate, mult, offset);
     });
     return ti_check_launch("gated_add_norm32");
 }

@@ -7,9 +7,10 @@ namespace ti {
 
 static inline int64_t ceil_div(int64_t a, int64_t b) { return (a + b - 1) / b; }
 
-PagedBook::PagedBook(int num_pages, int page_size, int window, int granule, int max_seqs, int max_pages_per_seq)
+PagedBook::PagedBook(int num_pages, int page_size, int window, int keep_first, int granule, int max_seqs, int max_pages_per_seq)
     : num_pages(num_pages), page_size(page_size), window(window), granule(std::max(1, granule)), max_seqs(max_seqs),
-      max_pages_per_seq(max_pages_per_seq), pages(num_pages), tables(max_seqs), first(max_seqs, 0),
+      max_pages_per_seq(max_pages_per_seq),
+      kept((int)ceil_div(ceil_div(std::max(0, keep_first), page_size), std::max(1, granule)) * std::max(1, granule)), pages(num_pages), tables(max_seqs), first(max_seqs, 0),
       host_table((size_t)max_seqs * max_pages_per_seq, 0) {}
 
 int PagedBook::pages_needed(int slot, int64_t new_length) const {
@@ -42,7 +43,7 @@ int PagedBook::first_needed_page(int64_t length) const {
 int PagedBook::release(int slot, int64_t length) {
     std::vector<int>& table = tables[slot];
     if (!window || table.empty()) return 0;
-    const int a = first[slot], b = std::min<int>(first_needed_page(length), (int)table.size());
+    const int a = std::max(first[slot], kept), b = std::min<int>(first_needed_page(length), (int)table.size());
     for (int i = a; i < b; ++i) {
         pages.give(table[i]);
         table[i] = -1;
@@ -54,7 +55,7 @@ int PagedBook::release(int slot, int64_t length) {
 int PagedBook::shrink(int slot, int64_t new_length) {
     std::vector<int>& table = tables[slot];
     const int keep = (int)ceil_div(new_length, page_size);
-    if (keep && first_needed_page(new_length) < first[slot])
+    if (keep && std::max(first_needed_page(new_length), kept) < first[slot])
         return ti_fail("cannot roll back to %lld positions: the pages of its window were given back", (long long)new_length), 2;
     for (int i = (int)table.size() - 1; i >= keep; --i)
         if (table[i] >= 0) pages.give(table[i]);
@@ -91,7 +92,7 @@ int64_t PagedBook::peak_pages(int n, const int* slots, const int64_t* counts, co
                 peak = std::max(peak, extra);
                 for (int s : touched) {
                     const int64_t b = std::min<int64_t>(first_needed_page(length[s]), logical[s]);
-                    extra -= std::max<int64_t>(0, b - first_now[s]);
+                    extra -= std::max<int64_t>(0, b - std::max(first_now[s], kept));
                     first_now[s] = (int)std::max<int64_t>(first_now[s], b);
                 }
                 touched.clear();
@@ -192,7 +193,7 @@ int CacheBook::truncate(int slot, int64_t length) {
         return ti_fail("cannot truncate a sequence of length %lld to %lld", (long long)lengths[slot], (long long)length), 2;
     if (has_state && length != lengths[slot]) return ti_fail("layers with a per-sequence state cannot roll back"), 2;
     for (PagedBook& g : groups)          // every group must be able to before any of them does
-        if (length > 0 && g.first_needed_page(length) < g.first[slot])
+        if (length > 0 && std::max(g.first_needed_page(length), g.kept) < g.first[slot])
             return ti_fail("cannot roll back to %lld positions: the pages of its window were given back", (long long)length), 2;
     for (PagedBook& g : groups)
         if (int rc = g.shrink(slot, length)) return rc;

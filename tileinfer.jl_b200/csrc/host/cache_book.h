@@ -18,19 +18,20 @@ struct PageWrite {
 
 class PagedBook {
 public:
-    PagedBook(int num_pages, int page_size, int window, int granule, int max_seqs, int max_pages_per_seq);
+    PagedBook(int num_pages, int page_size, int window, int keep_first, int granule, int max_seqs, int max_pages_per_seq);
     int pages_needed(int slot, int64_t new_length) const;
     int grow(int slot, int64_t new_length);                 // 0, or 2 with the text in ti_last_error()
-    int first_needed_page(int64_t length) const;
+    int first_needed_page(int64_t length) const;            // of the window; the kept pages before it are needed as well
     int release(int slot, int64_t length);
     int shrink(int slot, int64_t new_length);               // 0 or 2
     int64_t peak_pages(int n, const int* slots, const int64_t* counts, const std::vector<int64_t>& lengths, int64_t chunk_tokens) const;
     void flush(cudaStream_t stream);
 
     int num_pages, page_size, window, granule, max_seqs, max_pages_per_seq;
+    int kept;                                 // pages at a sequence's start that stay visible beside the window, in whole granules
     NumberPool pages;
     std::vector<std::vector<int>> tables;     // per slot: logical page index -> page, -1 once given back
-    std::vector<int> first;                   // per slot: first logical page still held
+    std::vector<int> first;                   // per slot: first logical page still held behind the kept ones
     std::vector<int32_t> host_table;          // [max_seqs][max_pages_per_seq], what the step planner reads
     std::vector<PageWrite> pending;           // table entries and fresh pages not yet written to the device
     // Where the device's copy of the block table and the value pool are (set once by the owner of the storage).

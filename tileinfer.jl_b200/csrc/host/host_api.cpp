@@ -24,9 +24,9 @@ extern "C" void* ti_cache_create(int max_seqs, long long max_seq_len, int has_st
     return c;
 }
 extern "C" void ti_cache_destroy(void* c) { delete (CacheBook*)c; }
-extern "C" int ti_cache_add_group(void* c, int num_pages, int page_size, int window, int granule, int max_pages_per_seq) {
+extern "C" int ti_cache_add_group(void* c, int num_pages, int page_size, int window, int keep_first, int granule, int max_pages_per_seq) {
     CacheBook* cache = (CacheBook*)c;
-    cache->groups.emplace_back(num_pages, page_size, window, granule, cache->max_seqs, max_pages_per_seq);
+    cache->groups.emplace_back(num_pages, page_size, window, keep_first, granule, cache->max_seqs, max_pages_per_seq);
     return (int)cache->groups.size() - 1;
 }
 // Where the group's block table and value pool live (device memory when on_device, else host memory).

@@ -3,7 +3,7 @@
 // (one "head" of kv_rank elements per position: pool[slot * kv_rank + i], slot = page * page_size + offset).
 //
 //   cq = T(a / rms(a) * wq),  a = row[0 : q_rank]
-//   c  = T(b / rms(b) * wkv), b = row[q_rank : q_rank + kv_rank]
+//   c  = T(b / rms(b) * wkv), b = row[q_rank : q_rank + kv_rank]          (q_rank 0: no query latent)
 //
 // With a rotated key part (rot > 0) the row has rot more elements after the two latents: one key part shared by all heads,
 // not normed, rotated by the position's angles (cos_sin [positions, rot / 2, 2] float; pairs (2i, 2i + 1) or (i, i + rot / 2)) in
@@ -41,7 +41,7 @@ __global__ void latent_inputs_kernel(const T* rows, size_t row_stride, const flo
     }
     sq = block_sum(sq, scratch);
     sk = block_sum(sk, scratch);
-    const float iq = 1.0f / sqrtf(sq / (float)q_rank + eps), ik = 1.0f / sqrtf(sk / (float)kv_rank + eps);
+    const float iq = q_rank > 0 ? 1.0f / sqrtf(sq / (float)q_rank + eps) : 0.f, ik = 1.0f / sqrtf(sk / (float)kv_rank + eps);
     const size_t slot = (size_t)__ldcg(slots + t);
     for (int i = threadIdx.x; i < normed; i += LI_THREADS) {
         if (i < q_rank) cq[(size_t)t * q_rank + i] = from_f32<T>(row[i] * iq * to_f32(wq[i]));
@@ -99,7 +99,7 @@ extern "C" int ti_latent_inputs(const void* rows, long long row_stride, const fl
                                 int q_rank, int kv_rank, int rot, const float* cos_sin, int interleaved, const int* positions, int pool_row,
                                 long long in_row, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return 0;
-    TI_REQUIRE(q_rank > 0 && kv_rank > 0 && rot >= 0 && q_rank + kv_rank + rot <= 12000, "latent_inputs: ranks %d and %d, %d rotated", q_rank, kv_rank, rot);
+    TI_REQUIRE(q_rank >= 0 && kv_rank > 0 && rot >= 0 && q_rank + kv_rank + rot <= 12000, "latent_inputs: ranks %d and %d, %d rotated", q_rank, kv_rank, rot);
     TI_REQUIRE((rows != nullptr) != (partials != nullptr), "latent_inputs: give rows or partial sums, not both");
     TI_REQUIRE(pool_row >= kv_rank + rot && in_row >= q_rank + kv_rank + rot, "latent_inputs: pool rows of %d for %d + %d", pool_row, kv_rank, rot);
     TI_REQUIRE(rot == 0 || (rot % 2 == 0 && cos_sin != nullptr && positions != nullptr), "latent_inputs: %d rotated elements need a table and positions", rot);

@@ -2,7 +2,8 @@
 //
 //   S_t = a_t S_(t-1) + b_t k_t v_t^T,   n_t = a_t n_(t-1) + b_t k_t,   o_t = S_t^T q_t
 //
-// (retention: a_t = the head's decay, b_t = 1, no n; the gated cell: a_t = keep, b_t = add). Instead of walking the tokens one by one, a
+// (retention: a_t = the head's decay, b_t = 1, no n; the gated cell: a_t = keep, b_t = add; the state-space cell: a_t = e^(l_t), b_t = dt_t, no
+// n, q and k shared by the heads of a group, and D_h v_t added to o_t). Instead of walking the tokens one by one, a
 // sequence's tokens of the step are cut into chunks of 64, counted from the step's first. With L_t the sum of ln a up to t inside a chunk
 // and S the state ahead of it,
 //
@@ -37,6 +38,10 @@ struct ChunkArgs {
     int B, H, D, V;
     const float* decay;          // [H], or null: coef [n, H, 2] = (keep, add)
     const float* coef;
+    int coef_log;                // coef holds (ln keep, add)
+    int vector;                  // there is a vector n beside S
+    int per_qk;                  // heads that share a q and a k
+    const float* skip;           // [H] or null: skip[h] * v joins o
     const float* cos_sin;        // [positions, rotary / 2, 2] or null
     int rotary;
     float q_scale, k_scale;
@@ -78,14 +83,16 @@ __device__ __forceinline__ void chunk_decays(const ChunkArgs& a, int h, int t0, 
     double l = 0.0;
     float b = 0.f;
     if (s < count) {
-        float keep = a.decay != nullptr ? a.decay[h] : 1.f;
+        float log_keep = 0.f;
         b = 1.f;
         if (a.coef != nullptr) {
             const float2 c = __ldcg(reinterpret_cast<const float2*>(a.coef) + (size_t)(t0 + s) * a.H + h);
-            keep = c.x;
+            log_keep = a.coef_log ? c.x : logf(c.x);
             b = c.y;
+        } else {
+            log_keep = logf(a.decay[h]);
         }
-        l = (double)fmaxf(logf(keep), -100.f);          // (e^-100 is zero beside anything 32-bit)
+        l = (double)fmaxf(log_keep, -100.f);          // (e^-100 is zero beside anything 32-bit)
     }
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -115,7 +122,7 @@ __device__ __forceinline__ void stage_qk(const ChunkArgs& a, float* dst, int off
             float* out = dst + s * MC_PITCH + d - d0;
             Vec16<T> v;
             if (s < count) {
-                const T* row = (const T*)a.rows + (size_t)(t0 + s) * a.ld + off + (size_t)h * D;
+                const T* row = (const T*)a.rows + (size_t)(t0 + s) * a.ld + off + (size_t)(h / a.per_qk) * D;
                 v.load_cg(row + d);
                 if (a.cos_sin != nullptr && d < a.rotary) {
                     const bool low = d < half;
@@ -142,7 +149,7 @@ __device__ __forceinline__ void stage_qk(const ChunkArgs& a, float* dst, int off
             const int s = e / width, d = d0 + e % width;
             float v = 0.f;
             if (s < count && d < D) {
-                const T* row = (const T*)a.rows + (size_t)(t0 + s) * a.ld + off + (size_t)h * D;
+                const T* row = (const T*)a.rows + (size_t)(t0 + s) * a.ld + off + (size_t)(h / a.per_qk) * D;
                 v = to_f32(__ldcg(row + d));
                 if (a.cos_sin != nullptr && d < a.rotary) {
                     const bool low = d < half;
@@ -234,7 +241,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_states_kernel(Chun
                     if (v + j < a.V) out[(size_t)d * a.V + v + j] = acc[i][4 * g + j];
         }
     }
-    if (a.coef != nullptr && v0 == 0 && threadIdx.x < MC_SLAB && d0 + threadIdx.x < a.D) {
+    if (a.vector && v0 == 0 && threadIdx.x < MC_SLAB && d0 + threadIdx.x < a.D) {
         float n = 0.f;
         for (int s = 0; s < count; ++s) n = fmaf(weight[s], ks[s * MC_PITCH + threadIdx.x], n);
         out[(size_t)a.D * a.V + d0 + threadIdx.x] = n;
@@ -245,7 +252,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_states_kernel(Chun
 template <int VEC>
 __global__ void __launch_bounds__(256) memory_chunk_scan_kernel(ChunkArgs a, float* state, long long state_stride, const int* seq_slots) {
     const int h = blockIdx.y, b = blockIdx.z;
-    const int DV = a.D * a.V, elements = DV + (a.coef != nullptr ? a.D : 0);
+    const int DV = a.D * a.V, elements = DV + (a.vector ? a.D : 0);
     const int e = (blockIdx.x * 256 + threadIdx.x) * VEC;
     pdl_enter();
     int first = 0;                                       // chunks of the sequences before this one: a warp counts 32 sequences at once
@@ -311,7 +318,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(Chu
     __shared__ double L[MC_TOKENS];
     __shared__ float add[MC_TOKENS], past[MC_TOKENS], den[MC_TOKENS];
     const int h = blockIdx.y, v0 = blockIdx.z * MC_SLAB, D = a.D, V = a.V;
-    const bool gated = a.coef != nullptr;
+    const bool gated = a.vector != 0;
     int t0 = 0, count = 0;
     pdl_enter();
     if (!chunk_of(a, blockIdx.x, t0, count)) return;
@@ -467,7 +474,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(Chu
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     const int c = (j < 4 ? 0 : 64) + cx * 4 + (j & 3);
-                    if (v0 + c < V) out.o[at + c] = acc[i][j];
+                    if (v0 + c < V) out.o[at + c] = a.skip != nullptr ? fmaf(a.skip[h], vs[t * MC_SLAB + c], acc[i][j]) : acc[i][j];
                 }
             continue;
         }
@@ -498,6 +505,38 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(Chu
     }
 }
 
+static int launch_chunks(const ChunkArgs& a, const ChunkOut& out, float* state, long long state_stride, int chunks, const int* seq_slots, int dtype,
+                         cudaStream_t stream) {
+    const int d_slabs = (a.D + MC_SLAB - 1) / MC_SLAB, v_slabs = (a.V + MC_SLAB - 1) / MC_SLAB;
+    const size_t smem_s = (size_t)MC_TOKENS * (MC_PITCH + MC_SLAB) * sizeof(float), smem_o = (size_t)MC_TOKENS * (2 * MC_PITCH + MC_SLAB) * sizeof(float);
+    const bool scan4 = a.D % 4 == 0 && (a.D * a.V) % 4 == 0 && state_stride % 4 == 0 && aligned16(state) && aligned16(a.ws);
+    const int elements = a.D * a.V + (a.vector ? a.D : 0);
+    TI_DISPATCH_DTYPE(dtype, {
+        constexpr int VEC = Vec16<T>::N;
+        const bool vectors = aligned16(a.rows) && a.ld % VEC == 0 && a.q_off % VEC == 0 && a.k_off % VEC == 0 && a.v_off % VEC == 0 && a.D % VEC == 0 && a.V % VEC == 0 &&
+                             (a.cos_sin == nullptr || ((a.rotary / 2) % VEC == 0 && aligned16(a.cos_sin)));
+        static bool configured = false;                  // per element type
+        if (!configured) {
+            cudaError_t e = cudaFuncSetAttribute(memory_chunk_states_kernel<T, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_s);
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(memory_chunk_states_kernel<T, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_s);
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(memory_chunk_outputs_kernel<T, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_o);
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(memory_chunk_outputs_kernel<T, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_o);
+            if (e != cudaSuccess) return ti_fail("memory_chunks: %s", cudaGetErrorString(e));
+            configured = true;
+        }
+        const dim3 grid_s(chunks, a.H, d_slabs * v_slabs), grid_o(chunks, a.H, v_slabs);
+        if (vectors) ti_launch(memory_chunk_states_kernel<T, true>, grid_s, dim3(MC_THREADS), smem_s, stream, a);
+        else ti_launch(memory_chunk_states_kernel<T, false>, grid_s, dim3(MC_THREADS), smem_s, stream, a);
+        if (int rc = ti_check_launch("memory_chunk_states")) return rc;
+        if (scan4) ti_launch(memory_chunk_scan_kernel<4>, dim3((elements / 4 + 255) / 256, a.H, a.B), dim3(256), 0, stream, a, state, state_stride, seq_slots);
+        else ti_launch(memory_chunk_scan_kernel<1>, dim3((elements + 255) / 256, a.H, a.B), dim3(256), 0, stream, a, state, state_stride, seq_slots);
+        if (int rc = ti_check_launch("memory_chunk_scan")) return rc;
+        if (vectors) ti_launch(memory_chunk_outputs_kernel<T, true>, grid_o, dim3(MC_THREADS), smem_o, stream, a, out);
+        else ti_launch(memory_chunk_outputs_kernel<T, false>, grid_o, dim3(MC_THREADS), smem_o, stream, a, out);
+    });
+    return ti_check_launch("memory_chunk_outputs");
+}
+
 // Floats of work space per (chunk, head).
 extern "C" int ti_memory_chunk_pitch(int D, int V) { return (D * V + D + 3) / 4 * 4; }
 
@@ -513,35 +552,21 @@ extern "C" int ti_memory_chunks(void* y, float* o, float* nq, const float* em, c
     TI_REQUIRE(coef == nullptr || (y != nullptr ? em != nullptr : nq != nullptr), "memory_chunks: the gated cell needs its divisor's pieces");
     TI_REQUIRE(H > 0 && D > 0 && V > 0 && H <= 65535 && B <= 65535, "memory_chunks: %d heads of %d x %d, %d sequences", H, D, V, B);
     TI_REQUIRE(cos_sin == nullptr || (positions != nullptr && rotary >= 2 && rotary % 2 == 0 && rotary <= D), "memory_chunks: rotation over %d of %d", rotary, D);
-    ChunkArgs a = {rows, ld, q_off, k_off, v_off, g_off, cu_seqlens, positions, B, H, D, V, decay, coef, cos_sin, cos_sin != nullptr ? rotary : 0,
-                   q_scale, k_scale, ws, ti_memory_chunk_pitch(D, V), total};
+    const ChunkArgs a = {rows, ld, q_off, k_off, v_off, g_off, cu_seqlens, positions, B, H, D, V, decay, coef, 0, coef != nullptr, 1, nullptr, cos_sin,
+                         cos_sin != nullptr ? rotary : 0, q_scale, k_scale, ws, ti_memory_chunk_pitch(D, V), total};
     const ChunkOut out = {y, o, nq, em, w, gate_sigmoid, eps};
-    const int d_slabs = (D + MC_SLAB - 1) / MC_SLAB, v_slabs = (V + MC_SLAB - 1) / MC_SLAB;
-    const size_t smem_s = (size_t)MC_TOKENS * (MC_PITCH + MC_SLAB) * sizeof(float), smem_o = (size_t)MC_TOKENS * (2 * MC_PITCH + MC_SLAB) * sizeof(float);
-    const bool scan4 = D % 4 == 0 && (D * V) % 4 == 0 && state_stride % 4 == 0 && aligned16(state) && aligned16(ws);
-    const int elements = D * V + (coef != nullptr ? D : 0);
-    TI_DISPATCH_DTYPE(dtype, {
-        constexpr int VEC = Vec16<T>::N;
-        const bool vectors = aligned16(rows) && ld % VEC == 0 && q_off % VEC == 0 && k_off % VEC == 0 && v_off % VEC == 0 && D % VEC == 0 && V % VEC == 0 &&
-                             (cos_sin == nullptr || ((rotary / 2) % VEC == 0 && aligned16(cos_sin)));
-        static bool configured = false;                  // per element type
-        if (!configured) {
-            cudaError_t e = cudaFuncSetAttribute(memory_chunk_states_kernel<T, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_s);
-            if (e == cudaSuccess) e = cudaFuncSetAttribute(memory_chunk_states_kernel<T, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_s);
-            if (e == cudaSuccess) e = cudaFuncSetAttribute(memory_chunk_outputs_kernel<T, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_o);
-            if (e == cudaSuccess) e = cudaFuncSetAttribute(memory_chunk_outputs_kernel<T, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_o);
-            if (e != cudaSuccess) return ti_fail("memory_chunks: %s", cudaGetErrorString(e));
-            configured = true;
-        }
-        const dim3 grid_s(chunks, H, d_slabs * v_slabs), grid_o(chunks, H, v_slabs);
-        if (vectors) ti_launch(memory_chunk_states_kernel<T, true>, grid_s, dim3(MC_THREADS), smem_s, stream, a);
-        else ti_launch(memory_chunk_states_kernel<T, false>, grid_s, dim3(MC_THREADS), smem_s, stream, a);
-        if (int rc = ti_check_launch("memory_chunk_states")) return rc;
-        if (scan4) ti_launch(memory_chunk_scan_kernel<4>, dim3((elements / 4 + 255) / 256, H, B), dim3(256), 0, stream, a, state, state_stride, seq_slots);
-        else ti_launch(memory_chunk_scan_kernel<1>, dim3((elements + 255) / 256, H, B), dim3(256), 0, stream, a, state, state_stride, seq_slots);
-        if (int rc = ti_check_launch("memory_chunk_scan")) return rc;
-        if (vectors) ti_launch(memory_chunk_outputs_kernel<T, true>, grid_o, dim3(MC_THREADS), smem_o, stream, a, out);
-        else ti_launch(memory_chunk_outputs_kernel<T, false>, grid_o, dim3(MC_THREADS), smem_o, stream, a, out);
-    });
-    return ti_check_launch("memory_chunk_outputs");
+    return launch_chunks(a, out, state, state_stride, chunks, seq_slots, dtype, stream);
+}
+
+// The state-space cell: rows [n, ld] of T with x (H * V columns) at x_off, B and C (groups * N each) at b_off and c_off; coef [n, H, 2] = (l, dt);
+// o [n, H * V] float = y with the skip in it. Work space as above.
+extern "C" int ti_ssm_chunks(float* o, const void* rows, long long ld, int x_off, int b_off, int c_off, float* state, long long state_stride,
+                             const float* coef, const float* skip, float* ws, float* total, int chunks, const int* cu_seqlens, const int* seq_slots,
+                             int B, int H, int groups, int N, int V, int dtype, cudaStream_t stream) {
+    if (B == 0 || chunks == 0) return 0;
+    TI_REQUIRE(H > 0 && groups > 0 && H % groups == 0 && N > 0 && V > 0 && H <= 65535 && B <= 65535, "ssm_chunks: %d heads in %d groups, %d x %d", H, groups, N, V);
+    const ChunkArgs a = {rows, ld, c_off, b_off, x_off, 0, cu_seqlens, nullptr, B, H, N, V, nullptr, coef, 1, 0, H / groups, skip, nullptr, 0, 1.f, 1.f, ws,
+                         ti_memory_chunk_pitch(N, V), total};
+    const ChunkOut out = {nullptr, o, nullptr, nullptr, nullptr, 0, 0.f};
+    return launch_chunks(a, out, state, state_stride, chunks, seq_slots, dtype, stream);
 }

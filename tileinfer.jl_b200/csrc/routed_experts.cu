@@ -87,7 +87,8 @@ extern "C" int ti_router_topk(const void* h, const void* wr, const float* logits
 
 // A router with more rules. z [n, ldz] holds the 32-bit logits of `total` = experts + pass choices (and, with a gate, one more
 // column: the gate's logit); without z the kernel computes them from h and wr (rows in that order). Per token:
-//   s = softmax(z[0 .. total)) (or sigmoid of each), c = s + correction (the CHOICE score; correction may be null);
+//   z += z_bias (which may be null);  s = softmax(z[0 .. total)) (or sigmoid of each), c = s + correction (the CHOICE score; correction may
+//   be null); with `softmax` 2 c = z itself and the weights are the softmax over the chosen logits alone;
 //   the choices form `groups` equal groups of neighbours, a group's score is its largest c (group_best 1) or the sum of its two
 //   largest (group_best 2), only the `keep` best groups stay
 //   (ties to the smaller index); of those the `top` largest c are chosen (ties to the smaller index);
@@ -97,8 +98,8 @@ extern "C" int ti_router_topk(const void* h, const void* wr, const float* logits
 // sigmoid(gate logit), or 1 without a gate.
 template <typename T>
 __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const float* z_in, long long ldz, int width, int experts, int total,
-                                     int softmax, const float* __restrict__ correction, int groups, int keep, int group_best, int top, int renormalize,
-                                     int always, int gate, int* __restrict__ ids, float* __restrict__ scores, float* __restrict__ pass_weight) {
+                                     int softmax, const float* __restrict__ z_bias, const float* __restrict__ correction, int groups, int keep, int group_best,
+                                     int top, int renormalize, int always, int gate, int* __restrict__ ids, float* __restrict__ scores, float* __restrict__ pass_weight) {
     __shared__ float z[RT_MAX_EXPERTS + 1], c[RT_MAX_EXPERTS], gs[RT_MAX_EXPERTS];
     __shared__ float scratch[33];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -117,7 +118,13 @@ __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const
         }
     }
     __syncthreads();
-    if (softmax) {
+    if (z_bias != nullptr) {
+        for (int e = threadIdx.x; e < total; e += RT_THREADS) z[e] += z_bias[e];
+        __syncthreads();
+    }
+    if (softmax == 2) {
+        // the choice and the weights rest on the logits themselves
+    } else if (softmax) {
         float m = -INFINITY;
         for (int e = threadIdx.x; e < total; e += RT_THREADS) m = fmaxf(m, z[e]);
         m = block_max(m, scratch);
@@ -174,6 +181,15 @@ __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const
             wsum += z[arg];
             __syncwarp();
         }
+        if (softmax == 2 && lane == 0) {                            // the chosen logits come largest first
+            const float m = scores[out];
+            wsum = 0.f;
+            for (int j = 0; j < top; ++j) {
+                const float v = expf(scores[out + j] - m);
+                scores[out + j] = v;
+                wsum += v;
+            }
+        }
         if (lane == 0) {
             const float div = renormalize ? wsum + 1e-20f : 1.0f;
             float pass = 0.f;
@@ -193,9 +209,10 @@ __global__ void router_select_kernel(const T* h, const T* __restrict__ wr, const
 }
 
 extern "C" int ti_router_select(const void* h, const void* wr, const float* z, long long ldz, int n, int width, int experts, int total, int softmax,
-                                const float* correction, int groups, int keep, int group_best, int top, int renormalize, int always, int gate, int* ids,
-                                float* scores, float* pass_weight, int dtype, cudaStream_t stream) {
+                                const float* z_bias, const float* correction, int groups, int keep, int group_best, int top, int renormalize, int always,
+                                int gate, int* ids, float* scores, float* pass_weight, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
+    TI_REQUIRE(softmax != 2 || (correction == nullptr && keep == groups && renormalize), "router_select: a choice on the logits has no correction and no groups");
     TI_REQUIRE(experts >= 0 && total >= experts && total >= 1 && total <= RT_MAX_EXPERTS && top >= 1 && top <= total && always >= 0,
                "router_select: top %d of %d choices (%d experts)", top, total, experts);
     TI_REQUIRE(groups >= 1 && total % groups == 0 && keep >= 1 && keep <= groups && keep * (total / groups) >= top,
@@ -203,7 +220,7 @@ extern "C" int ti_router_select(const void* h, const void* wr, const float* z, l
     TI_REQUIRE(group_best == 1 || group_best == 2, "router_select: a group's score from its %d best", group_best);
     TI_REQUIRE(total == experts || pass_weight != nullptr, "router_select: pass choices need their weights' output");
     TI_DISPATCH_DTYPE(dtype, (ti_launch(router_select_kernel<T>, dim3(n), dim3(RT_THREADS), 0, stream, (const T*)h, (const T*)wr, z, ldz, width, experts,
-                                        total, softmax, correction, groups, keep, group_best, top, renormalize, always, gate, ids, scores, pass_weight)));
+                                        total, softmax, z_bias, correction, groups, keep, group_best, top, renormalize, always, gate, ids, scores, pass_weight)));
     return ti_check_launch("router_select");
 }
 

@@ -295,25 +295,28 @@ SHORT_PROMPT = 384
 SHORT_STEP = 512
 
 
-def attention(out, q, cache, meta, step, spec, sink=None, chunk=0, distance_bias2=None, cap=0.0, slopes2=None) -> bool:
+def attention(out, q, cache, meta, step, spec, sink=None, chunk=0, distance_bias2=None, cap=0.0, slopes2=None, keep=0) -> bool:
     """``sink`` [heads] float32: one more term exp(sink[head]) in every softmax's denominator. ``chunk`` > 0: a key is visible only
     inside the query's chunk of so many positions; ``distance_bias2`` [heads, L] float32: the bias by distance times log2(e) (the
     kernels work in base 2), entry min(distance, L - 1). ``cap`` > 0: the scaled score s becomes cap tanh(s / cap) first; ``slopes2``
-    [heads] float32: a slope by distance taken off, times log2(e)."""
+    [heads] float32: a slope by distance taken off, times log2(e). ``keep``: beside a window, the first ``keep`` positions stay visible."""
     if q.dtype != torch.bfloat16:
         return False
     # The entry points with a sink take it as one more argument before the stream; without a sink the plain ones are called.
     extra = (sink.data_ptr(),) if sink is not None else ()
     L = lib()
     shaped = bool(cap) or slopes2 is not None
-    ruled = bool(chunk) or distance_bias2 is not None or shaped
+    ruled = bool(chunk) or distance_bias2 is not None or shaped or bool(keep)
     if ruled:
         extra = (sink.data_ptr() if sink is not None else None, int(chunk or 0), distance_bias2.data_ptr() if distance_bias2 is not None else None,
                  distance_bias2.shape[1] if distance_bias2 is not None else 0)
         decode_fn, tc_fn, mma_fn = L.ti_attention_decode_biased, L.ti_attention_prefill_tc_biased, L.ti_attention_prefill_biased
-        if shaped:
+        if shaped or keep:
             extra += (float(cap), slopes2.data_ptr() if slopes2 is not None else None)
             decode_fn, tc_fn, mma_fn = L.ti_attention_decode_ruled, L.ti_attention_prefill_tc_ruled, L.ti_attention_prefill_ruled
+        if keep:
+            extra += (int(keep),)
+            decode_fn, tc_fn, mma_fn = L.ti_attention_decode_kept, L.ti_attention_prefill_tc_kept, L.ti_attention_prefill_kept
     else:
         decode_fn, tc_fn, mma_fn = ((L.ti_attention_decode_sink, L.ti_attention_prefill_tc_sink, L.ti_attention_prefill_sink) if sink is not None
                                     else (L.ti_attention_decode_shared, L.ti_attention_prefill_tc, L.ti_attention_prefill))

@@ -18,7 +18,7 @@ _DECLS = {
     "ti_pool_give": (c_int, [c_void_p, c_int]), "ti_pool_free": (c_int, [c_void_p]), "ti_pool_held": (c_int, [c_void_p]),
     "ti_pool_is_held": (c_int, [c_void_p, c_int]),
     "ti_cache_create": (c_void_p, [c_int, c_longlong, c_int]), "ti_cache_destroy": (None, [c_void_p]),
-    "ti_cache_add_group": (c_int, [c_void_p, c_int, c_int, c_int, c_int, c_int]),
+    "ti_cache_add_group": (c_int, [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int]),
     "ti_cache_group_storage": (None, [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_longlong, c_int]),
     "ti_cache_alloc_slot": (c_int, [c_void_p]), "ti_cache_free_slot": (c_int, [c_void_p, c_int]),
     "ti_cache_length": (c_longlong, [c_void_p, c_int]), "ti_cache_lengths": (None, [c_void_p, c_int, _INTS, _LONGS]),

@@ -81,6 +81,7 @@ _SIGNATURES = {
     "ti_attention_plain": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "ti_attention_plain_biased": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _I, _P],
     "ti_attention_plain_ruled": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _F, _P, _I, _P],
+    "ti_attention_plain_kept": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _F, _P, _I, _I, _P],
     "ti_gemm_plain": [_P, _L, _P, _L, _P, _I, _I, _I, _I, _F, _F, _F, _F, _I, _P],
     "ti_argmax": [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P],
     "ti_sample": [_P, _L, _I, _I, _F, _I, _F, _P, _P, _P, _P, _P],
@@ -90,7 +91,7 @@ _SIGNATURES = {
 }
 
 
-_KERNELS_PER_CALL = {"ti_memory_chunks": 3}
+_KERNELS_PER_CALL = {"ti_memory_chunks": 3, "ti_ssm_chunks": 3}
 
 
 def lib():
@@ -172,6 +173,8 @@ _SIGNATURES_FAST["ti_attention_decode_biased"] = _SIGNATURES_FAST["ti_attention_
 # ... and with a cap of the scores and a slope per head after those
 for _name in ("prefill", "prefill_tc", "decode"):
     _SIGNATURES_FAST[f"ti_attention_{_name}_ruled"] = _SIGNATURES_FAST[f"ti_attention_{_name}_biased"][:-1] + [_F, _P, _P]
+    # ... and with a number of first positions that stay visible beside the window
+    _SIGNATURES_FAST[f"ti_attention_{_name}_kept"] = _SIGNATURES_FAST[f"ti_attention_{_name}_ruled"][:-1] + [_I, _P]
 _SIGNATURES_FAST["ti_attention_prefill_tc_sink"] = _SIGNATURES_FAST["ti_attention_prefill_tc"][:-1] + [_P, _P]
 _SIGNATURES.update(_SIGNATURES_FAST)
 
@@ -201,11 +204,11 @@ _SIGNATURES.update({
     "ti_lightning_scan": [_P, _P, _L, _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "ti_lightning_out": [_P, _P, _P, _L, _P, _F, _I, _I, _I, _P],
     "ti_conv_attention_inputs": [_P, _L, _P, _P, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I,
-                                 _I, _I, _I, _P],
+                                 _I, _I, _I, _I, _I, _P],
     "ti_conv_state_update": [_P, _P, _L, _P, _I, _P, _P, _I, _I, _I, _P],
     "ti_sigmoid_gate": [_P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P],
     "ti_sum_add_norm32": [_P, _P, _P, _I, _L, _P, _P, _I, _L, _P, _P, _I, _F, _I, _I, _I, _P],
-    "ti_router_select": [_P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P],
+    "ti_router_select": [_P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P],
     "ti_gated_act": [_P, _P, _I, _I, _I, _I, _P],
 })
 
@@ -234,7 +237,7 @@ _SIGNATURES.update({
 
 # Gated additions to a stream normed in groups, a convolution over a step's rows; retention and the gated matrix memory.
 _SIGNATURES.update({
-    "ti_gated_add_norm32": [_P, _P, _P, _I, _L, _P, _P, _I, _P, _P, _P, _I, _L, _P, _P, _P, _F, _I, _P, _I, _P, _L, _P, _P, _I, _I, _I, _P],
+    "ti_gated_add_norm32": [_P, _P, _P, _I, _L, _P, _P, _I, _P, _P, _P, _I, _L, _P, _F, _P, _P, _I, _F, _I, _P, _I, _P, _L, _P, _P, _I, _I, _I, _P],
     "ti_conv_rows": [_P, _P, _P, _I, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "ti_retention_scan": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _I, _P, _F, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "ti_memory_gates": [_P, _P, _P, _L, _P, _F, _P, _L, _P, _P, _I, _I, _P],
@@ -242,4 +245,12 @@ _SIGNATURES.update({
     "ti_memory_chunks": [_P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P, _L, _P, _P, _P, _I, _P, _F, _F, _P, _I, _F, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     "ti_memory_token": [_P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P, _L, _P, _P, _L, _P, _F, _P, _I, _P, _F, _F, _P, _I, _F, _P, _I, _I, _I, _I,
                         _I, _P],
+})
+
+# The state-space recurrence: inputs, one-token step, chunks of a prompt, gate and norm of its output.
+_SIGNATURES.update({
+    "ti_ssm_inputs": [_P, _P, _P, _L, _I, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ti_ssm_token": [_P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "ti_ssm_chunks": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ti_ssm_gate_norm": [_P, _P, _P, _L, _P, _F, _I, _I, _I, _I, _P],
 })

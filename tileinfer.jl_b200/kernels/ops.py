@@ -133,14 +133,15 @@ def attention_inputs(qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, eps, rota
 
 
 def attention_plain(out, q, k_cache, v_cache, block_table, tok_slot, positions, scale, nq, nkv, head_dim,
-                    page_size, window=0, sink=None, chunk=0, distance_bias=None, cap=0.0, slopes=None):
+                    page_size, window=0, sink=None, chunk=0, distance_bias=None, cap=0.0, slopes=None, keep=0):
     """``sink`` [nq] float32: one more term exp(sink[head]) in every softmax's denominator (no key, no value). ``chunk`` > 0: a
     key is visible only inside the query's chunk of so many positions (counted from the sequence's start). ``distance_bias``
     [nq, L] float32: entry [head, min(distance, L - 1)] is added to the scaled score. ``cap`` > 0: the scaled score s becomes
-    cap tanh(s / cap) before that; ``slopes`` [nq] float32: slopes[head] * distance is taken off."""
+    cap tanh(s / cap) before that; ``slopes`` [nq] float32: slopes[head] * distance is taken off. ``keep``: beside a
+    window, the sequence's first ``keep`` positions stay visible."""
     if sink is not None:
         _need(sink, "sink", torch.float32)
-    if cap or slopes is not None:
+    if cap or slopes is not None or keep:
         for t, name in ((slopes, "slopes"), (distance_bias, "distance_bias")):
             if t is not None:
                 _need(t, name, torch.float32)
@@ -148,11 +149,11 @@ def attention_plain(out, q, k_cache, v_cache, block_table, tok_slot, positions, 
                     raise KernelError(f"attention: {name} {tuple(t.shape)} for {nq} heads")
         _need(out, "out"); _need(q, "q", out.dtype); _need(k_cache, "k_cache", out.dtype); _need(v_cache, "v_cache", out.dtype)
         _need(block_table, "block_table", torch.int32); _need(tok_slot, "tok_slot", torch.int32); _need(positions, "positions", torch.int32)
-        check(lib().ti_attention_plain_ruled(out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(),
+        check(lib().ti_attention_plain_kept(out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(),
                                              block_table.stride(0), tok_slot.data_ptr(), positions.data_ptr(), scale, q.shape[0], nq, nkv,
                                              head_dim, page_size, window or 0, _ptr(sink), int(chunk or 0), _ptr(distance_bias),
-                                             distance_bias.shape[1] if distance_bias is not None else 0, cap, _ptr(slopes), dtype_code(out.dtype),
-                                             _stream()), "attention_plain")
+                                             distance_bias.shape[1] if distance_bias is not None else 0, cap, _ptr(slopes), int(keep),
+                                             dtype_code(out.dtype), _stream()), "attention_plain")
         return
     if chunk or distance_bias is not None:
         if distance_bias is not None:
@@ -349,28 +350,31 @@ def latent_inputs(rows, cq, pool, wq, wkv, eps, slots, q_rank, kv_rank, rotation
     """rows [n, >= q_rank + kv_rank] (or 32-bit partial sums [s, n, ...]) -> cq [n, q_rank] and the key/value latent of every
     token at its place ``slots[t]`` of ``pool`` [positions, pool_row]; both RMS-normed in 32-bit with plain weights. With
     ``rotation`` the rotary_dim elements after the latents are a key part shared by all heads: rotated by ``positions`` and
-    written behind the latent in the pool's row (``pool_row`` >= kv_rank + rotary_dim elements, zeros after)."""
+    written behind the latent in the pool's row (``pool_row`` >= kv_rank + rotary_dim elements, zeros after). ``q_rank`` 0: no query
+    latent (``cq`` and ``wq`` None)."""
     rot = int(rotation.rotary_dim) if rotation is not None else 0
     pool_row = int(pool_row or kv_rank)
     if rotation is not None:
         _need(rotation.cos_sin, "cos_sin", torch.float32); _need(positions, "positions", torch.int32)
         if rotation.cos_sin.shape[1] * 2 != rot:
             raise KernelError(f"latent_inputs: {rot} rotated elements with a table of {tuple(rotation.cos_sin.shape)}")
-    _need(cq, "cq"); _need(pool, "pool", cq.dtype); _need(wq, "wq", cq.dtype); _need(wkv, "wkv", cq.dtype); _need(slots, "slots", torch.int32)
+    _need(pool, "pool"); _need(wkv, "wkv", pool.dtype); _need(slots, "slots", torch.int32)
+    if q_rank:
+        _need(cq, "cq", pool.dtype); _need(wq, "wq", pool.dtype)
     if rows.dim() == 3:
         _need(rows, "partial sums", torch.float32)
         args = (None, 0, rows.data_ptr(), rows.shape[0], rows.stride(0))
         n, in_row = rows.shape[1], rows.shape[2]
     else:
-        _need(rows, "rows", cq.dtype, contiguous=False)
+        _need(rows, "rows", pool.dtype, contiguous=False)
         if rows.stride(1) != 1:
             raise KernelError("latent_inputs: rows must be dense")
         args = (rows.data_ptr(), rows.stride(0), None, 0, 0)
         n, in_row = rows.shape[0], rows.shape[1]
-    check(lib().ti_latent_inputs(*args, cq.data_ptr(), pool.data_ptr(), wq.data_ptr(), wkv.data_ptr(), eps, slots.data_ptr(), n,
+    check(lib().ti_latent_inputs(*args, _ptr(cq), pool.data_ptr(), _ptr(wq), wkv.data_ptr(), eps, slots.data_ptr(), n,
                                  q_rank, kv_rank, rot, _ptr(rotation.cos_sin) if rotation is not None else None,
                                  int(bool(rotation.interleaved)) if rotation is not None else 0, _ptr(positions), pool_row, in_row,
-                                 dtype_code(cq.dtype), _stream()), "latent_inputs")
+                                 dtype_code(pool.dtype), _stream()), "latent_inputs")
 
 
 def head_gemm(y, x, w):
@@ -472,6 +476,8 @@ def expert_combine(out, y, pair_row, scores, shared, top, scale_output=False, h=
     _need(out, "out"); _need(y, "y", out.dtype); _need(pair_row, "pair_row", torch.int32); _need(scores, "scores", torch.float32)
     if shared is not None:
         _need(shared, "shared", out.dtype)
+    if logit_bias is not None:
+        _need(logit_bias, "logit_bias", torch.float32)
     if pass_weight is not None:
         _need(pass_weight, "pass_weight", torch.float32); _need(h, "h", out.dtype)
     n, width = out.shape
@@ -528,23 +534,22 @@ def lightning_out(y, o, gate, w, eps):
 
 
 def conv_attention_inputs(rows, bias, conv, taps, state, q_norm_w, k_norm_w, eps, rotation, q_out, k_cache, v_cache, step, slot_map,
-                          nq, nkv, dim, vdim, padded, page_size, write_kv=True, head_norm=False, shared_kv=False):
+                          nq, nkv, dim, vdim, padded, page_size, write_kv=True, head_norm=False, shared_kv=False, norm_last=False):
     """The step's projected rows (queries, then keys and values with ``write_kv``) -> bias, causal convolution over time (history
     from ``state`` [slots, taps - 1, channels] float32), whole-row RMS norms of q and k (``head_norm``: every head by itself, with
-    one weight of the head's size), rotation (``shared_kv``: no value rows, the values are the keys' rows before norm and rotation) -> q_out [n, nq, padded] and the keys and values at ``slot_map`` in the pools. ``step``
+    one weight of the head's size; ``norm_last``: after the rotation instead of before it), rotation (``shared_kv``: no value rows, the values are the keys' rows before norm and rotation) -> q_out [n, nq, padded] and the keys and values at ``slot_map`` in the pools. ``step``
     gives positions, cu_seqlens, seq_slots, kv_lens."""
     _need(rows, "rows", q_out.dtype, contiguous=False); _need(q_out, "q_out")
     cos_sin = rotation.cos_sin if rotation is not None else None
     rotary = int(rotation.rotary_dim) if rotation is not None else 0
-    if rotation is not None and rotation.interleaved:
-        raise KernelError("conv_attention_inputs: only the half-split pairing is built")
     if state is not None:
         _need(state, "state", torch.float32)
     check(lib().ti_conv_attention_inputs(rows.data_ptr(), rows.stride(0), _ptr(bias), _ptr(conv), taps, _ptr(state), _ptr(q_norm_w), _ptr(k_norm_w),
                                          eps, _ptr(cos_sin), rotary, q_out.data_ptr(), _ptr(k_cache), _ptr(v_cache), step.positions.data_ptr(),
                                          _ptr(slot_map), step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), step.kv_lens.data_ptr(),
                                          rows.shape[0], step.n_seqs, nq, nkv, dim, vdim, padded, page_size, int(bool(write_kv)),
-                                         int(bool(head_norm)), int(bool(shared_kv)), dtype_code(q_out.dtype), _stream()), "conv_attention_inputs")
+                                         int(bool(head_norm)), int(bool(shared_kv)), int(bool(rotation is not None and rotation.interleaved)),
+                                         int(bool(norm_last)), dtype_code(q_out.dtype), _stream()), "conv_attention_inputs")
 
 
 def conv_state_update(state, rows, bias, taps, step, channels):
@@ -565,10 +570,11 @@ def sigmoid_gate(y, attn, gate, heads, vdim, padded, per_head=False):
 
 
 def router_select(h, wr, logits, experts, total, top, ids, scores, pass_weight=None, softmax=True, correction=None, groups=1, keep=1,
-                  group_best=1, renormalize=True, always=0, gate=False):
+                  group_best=1, renormalize=True, always=0, gate=False, logit_bias=None, on_logits=False):
     """The router with groups, a correction for the choice, normalised weights, pass-through choices and a gated always-on unit
     (``csrc/routed_experts.cu``: router_select). ``group_best`` 1 or 2: a group's score is its best choice score or the sum of its two
-    best. ``logits`` [n, >= total (+ 1 with gate)] float32 or None (then from h and wr)."""
+    best. ``logit_bias`` [total] float32 is added to the logits; ``on_logits``: the largest logits are chosen and weighted by the softmax over
+    them. ``logits`` [n, >= total (+ 1 with gate)] float32 or None (then from h and wr)."""
     _need(h, "h"); _need(wr, "wr", h.dtype); _need(ids, "ids", torch.int32); _need(scores, "scores", torch.float32)
     n, width = h.shape
     if tuple(ids.shape) != (n, top + always) or ids.shape != scores.shape or wr.shape[0] != total + int(bool(gate)):
@@ -577,10 +583,12 @@ def router_select(h, wr, logits, experts, total, top, ids, scores, pass_weight=N
         _need(logits, "logits", torch.float32, contiguous=False)
     if correction is not None:
         _need(correction, "correction", torch.float32)
+    if logit_bias is not None:
+        _need(logit_bias, "logit_bias", torch.float32)
     if pass_weight is not None:
         _need(pass_weight, "pass_weight", torch.float32)
     check(lib().ti_router_select(h.data_ptr(), wr.data_ptr(), _ptr(logits), logits.stride(0) if logits is not None else 0, n, width, experts, total,
-                                 int(bool(softmax)), _ptr(correction), groups, keep, group_best, top, int(bool(renormalize)), always, int(bool(gate)),
+                                 2 if on_logits else int(bool(softmax)), _ptr(logit_bias), _ptr(correction), groups, keep, group_best, top, int(bool(renormalize)), always, int(bool(gate)),
                                  ids.data_ptr(), scores.data_ptr(), _ptr(pass_weight), dtype_code(h.dtype), _stream()), "router_select")
 
 
@@ -740,9 +748,10 @@ def _branch_args(d, dtype, name):
     return (d.data_ptr(), None, 0, d.stride(0))
 
 
-def gated_add_norm32(x, d, gate, h, w, eps, groups=1, d_bias=None, gate_bias=None, index=None, scores=None, conv=None):
-    """x += (d + d_bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``d`` None: x stays as it is; ``gate`` None: no gate), then
-    h = x normed by its root mean square in ``groups`` equal parts, times w. ``d``: rows [n, size], 32-bit partial sums [s, n, size], or
+def gated_add_norm32(x, d, gate, h, w, eps, groups=1, d_bias=None, gate_bias=None, index=None, scores=None, conv=None, mult=1.0,
+                     offset=False):
+    """x += mult * (d + d_bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``d`` None: x stays as it is; ``gate`` None: no gate), then
+    h = x normed by its root mean square in ``groups`` equal parts, times w (``offset``: times 1 + w). ``d``: rows [n, size], 32-bit partial sums [s, n, size], or
     with ``index`` and ``scores`` [n, per_row] rows still apart, of which row t's are added up. ``conv`` (weights [taps, size], history view
     [slots, >= (taps - 1) * size] float32 or None, seq_slots, out): one-token steps only, out = h + conv(h), the history moved on."""
     _need(x, "x", torch.float32); _need(h, "h"); _need(w, "w", h.dtype)
@@ -757,7 +766,7 @@ def gated_add_norm32(x, d, gate, h, w, eps, groups=1, d_bias=None, gate_bias=Non
     if index is not None:
         _need(index, "index", torch.int32); _need(scores, "scores", torch.float32)
     check(lib().ti_gated_add_norm32(x.data_ptr(), *_branch_args(d, h.dtype, "d"), _ptr(index), _ptr(scores), index.shape[1] if index is not None else 0,
-                                    _ptr(d_bias), *_branch_args(gate, h.dtype, "gate"), _ptr(gate_bias), h.data_ptr(), w.data_ptr(), eps, groups, *c,
+                                    _ptr(d_bias), *_branch_args(gate, h.dtype, "gate"), _ptr(gate_bias), mult, h.data_ptr(), w.data_ptr(), int(bool(offset)), eps, groups, *c,
                                     n, size, dtype_code(h.dtype), _stream()), "gated_add_norm32")
 
 
@@ -846,3 +855,56 @@ def memory_chunks(rows, offs, state, step, heads, dim, vdim, ws, total, chunks, 
                                  _ptr(coef), *_rotation_args(rotation, step), q_scale, k_scale, _ptr(w), int(bool(gate_sigmoid)), eps, ws.data_ptr(),
                                  total.data_ptr(), chunks, step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), step.n_seqs, heads, dim, vdim,
                                  dtype_code(rows.dtype), _stream()), "memory_chunks")
+
+
+# ---------------------------------------------------------------- the state-space recurrence
+def ssm_inputs(xbc, coef, rows, x_off, dt_off, conv, bias, hist, dt_bias, a_log, step):
+    """rows [n, ld]: x | B | C (as many columns as ``xbc`` has) from ``x_off``, dt' from ``dt_off`` -> xbc = SiLU(causal convolution + bias), conv
+    [taps, channels], earlier rows from ``hist`` [slots, >= (taps - 1) * channels] float32 (None with one tap); coef [n, heads, 2] float32 =
+    (-exp(a_log) dt, dt), dt = softplus(dt' + dt_bias). In one-token steps the history moves on, else ``history_update`` does that."""
+    _need(xbc, "xbc"); _need(coef, "coef", torch.float32); _need(rows, "rows", xbc.dtype, contiguous=False); _need(conv, "conv", xbc.dtype)
+    _need(bias, "bias", xbc.dtype); _need(dt_bias, "dt_bias", torch.float32); _need(a_log, "a_log", torch.float32)
+    if hist is not None:
+        _need(hist, "history", torch.float32, contiguous=False)
+    n, channels = xbc.shape
+    heads = dt_bias.numel()
+    if tuple(conv.shape[1:]) != (channels,) or bias.numel() != channels or a_log.numel() != heads or tuple(coef.shape) != (n, heads, 2):
+        raise KernelError(f"ssm_inputs: conv {tuple(conv.shape)}, bias {tuple(bias.shape)}, coef {tuple(coef.shape)} for {channels} channels")
+    if max(x_off + channels, dt_off + heads) > rows.shape[1]:
+        raise KernelError(f"ssm_inputs: columns {x_off} + {channels} and {dt_off} + {heads} in rows of {rows.shape[1]}")
+    check(lib().ti_ssm_inputs(xbc.data_ptr(), coef.data_ptr(), rows.data_ptr(), rows.stride(0), x_off, dt_off, conv.data_ptr(), conv.shape[0],
+                              bias.data_ptr(), _ptr(hist), hist.stride(0) if hist is not None else 0, dt_bias.data_ptr(), a_log.data_ptr(),
+                              step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), n, step.n_seqs, channels, heads, int(bool(step.is_decode)),
+                              dtype_code(xbc.dtype), _stream()), "ssm_inputs")
+
+
+def ssm_token(y, xbc, coef, skip, state, step, heads, groups, dim, vdim):
+    """One token per sequence: S = e^l S + dt B x^T, y = S^T C + skip x. xbc [n, heads * vdim + 2 * groups * dim]; ``state`` [slots, >= heads * dim *
+    vdim] float32; y [n, heads * vdim] float32."""
+    _need(y, "y", torch.float32); _need(xbc, "xbc"); _need(coef, "coef", torch.float32); _need(skip, "skip", torch.float32)
+    _need(state, "state", torch.float32, contiguous=False)
+    if xbc.shape[1] != heads * vdim + 2 * groups * dim or state.shape[1] < heads * dim * vdim:
+        raise KernelError(f"ssm_token: rows of {xbc.shape[1]}, states of {state.shape[1]} for {heads} heads of {dim} x {vdim} in {groups} groups")
+    check(lib().ti_ssm_token(y.data_ptr(), xbc.data_ptr(), coef.data_ptr(), skip.data_ptr(), state.data_ptr(), state.stride(0), step.seq_slots.data_ptr(),
+                             step.n_seqs, xbc.shape[1], heads, groups, dim, vdim, dtype_code(xbc.dtype), _stream()), "ssm_token")
+
+
+def ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, total, chunks):
+    """The same over a step's tokens in chunks of CHUNK_TOKENS. ``ws``, ``total`` [chunks, heads]: float32 work space (``memory_chunk_sizes``)."""
+    _need(y, "y", torch.float32); _need(xbc, "xbc"); _need(coef, "coef", torch.float32); _need(skip, "skip", torch.float32)
+    for t, name in ((state, "state"), (ws, "ws"), (total, "total")):
+        _need(t, name, torch.float32, contiguous=False)
+    if xbc.shape[1] != heads * vdim + 2 * groups * dim or state.shape[1] < heads * dim * vdim:
+        raise KernelError(f"ssm_chunks: rows of {xbc.shape[1]}, states of {state.shape[1]} for {heads} heads of {dim} x {vdim} in {groups} groups")
+    if ws.numel() < chunks * heads * int(lib().ti_memory_chunk_pitch(dim, vdim)) or total.numel() < chunks * heads:
+        raise KernelError(f"ssm_chunks: work space of {ws.numel()} floats for {chunks} chunks")
+    check(lib().ti_ssm_chunks(y.data_ptr(), xbc.data_ptr(), xbc.shape[1], 0, heads * vdim, heads * vdim + groups * dim, state.data_ptr(), state.stride(0),
+                              coef.data_ptr(), skip.data_ptr(), ws.data_ptr(), total.data_ptr(), chunks, step.cu_seqlens.data_ptr(),
+                              step.seq_slots.data_ptr(), step.n_seqs, heads, groups, dim, vdim, dtype_code(xbc.dtype), _stream()), "ssm_chunks")
+
+
+def ssm_gate_norm(out, y, z, w, eps, parts):
+    """out = (y * SiLU(z)), the row in ``parts`` equal parts each divided by its own root mean square, times w. y float32, z rows may be strided."""
+    _need(out, "out"); _need(y, "y", torch.float32); _need(z, "z", out.dtype, contiguous=False); _need(w, "w", out.dtype)
+    check(lib().ti_ssm_gate_norm(out.data_ptr(), y.data_ptr(), z.data_ptr(), z.stride(0), w.data_ptr(), eps, parts, out.shape[0], out.shape[1],
+                                 dtype_code(out.dtype), _stream()), "ssm_gate_norm")

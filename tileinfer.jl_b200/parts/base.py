@@ -46,8 +46,8 @@ from ..config.spec import TensorDecl
 class CacheRequest:
     """Per-sequence storage a mixer needs for one layer.
 
-    ``kind == "paged_kv"``: keys and values of every position (or of the last ``window``),
-    ``kv_heads × head_dim`` each, in pages. ``kind == "state"``: a tensor of fixed ``shape``
+    ``kind == "paged_kv"``: keys and values of every position (or of the last ``window`` and the first
+    ``keep_first``), ``kv_heads × head_dim`` each, in pages. ``kind == "state"``: a tensor of fixed ``shape``
     and ``dtype`` per sequence, zeroed when a sequence starts. Any other kind is one that was
     registered with ``cache.register_cache_kind``; its group class reads what it needs from these fields.
     """
@@ -57,9 +57,10 @@ class CacheRequest:
     window: Optional[int] = None
     shape: Tuple[int, ...] = ()
     dtype: Optional[torch.dtype] = None          # None: the model's element type
+    keep_first: int = 0
 
     def group_key(self):
-        return (self.kind, self.kv_heads, self.head_dim, self.window, tuple(self.shape), self.dtype)
+        return (self.kind, self.kv_heads, self.head_dim, self.window, tuple(self.shape), self.dtype, self.keep_first)
 
 
 class Part:

@@ -3,7 +3,8 @@ h = norm1(x), on a 32-bit stream.
 ``post_norm``: x += m norm1(mixer(x)); x += m norm2(ffn(x)); x += m token_input(x), on a 32-bit stream.
 ``sandwich``: x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))), on a 32-bit stream.
 ``hyper``: pre-norm sublayers that read, rewrite and write to several copies of a 32-bit stream through learned tables.
-``gated``: pre-norm sublayers added to a 32-bit stream through learned gates, with a short causal convolution ahead of the mixer.
+``gated``: pre-norm sublayers added to a 32-bit stream, where asked through learned gates, times a constant, and with a short causal
+convolution ahead of the mixer.
 
 Each residual add is fused with the norm that follows it, so a block receives the already
 normed input ``h`` and produces the next block's normed input with ``next_norm`` (the next
@@ -243,13 +244,13 @@ class ConvolvedRead:
     def forward(self, x, out):
         return self.gated_add(x, None, out)
 
-    def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None):
+    def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None, mult=1.0):
         taps, size = self.conv.shape
         hist = self.cache.state.view(self.cache.state.shape[0], -1) if taps > 1 else None
         convolved = self.rt.buffer(self.OUT, tuple(out.shape))
         if self.step.is_decode:
-            return self.norm.gated_add(x, delta, out, gate, bias, gate_bias, conv=(self.conv, hist, self.step.seq_slots, convolved))
-        self.norm.gated_add(x, delta, out, gate, bias, gate_bias)
+            return self.norm.gated_add(x, delta, out, gate, bias, gate_bias, conv=(self.conv, hist, self.step.seq_slots, convolved), mult=mult)
+        self.norm.gated_add(x, delta, out, gate, bias, gate_bias, mult=mult)
         ops.conv_rows(convolved, out, self.conv, hist, self.step)
         if taps > 1:
             ops.history_update(hist, out, taps, self.step, size)
@@ -260,10 +261,10 @@ class ConvolvedRead:
 class GatedBlock(Part):
     """Pre-norm sublayers on a 32-bit stream, each multiplied by a gate before it is added (a layer may have no feed-forward):
 
-        h = norm1(x);   x += mixer(h + conv(h)) * sigmoid(R1 h + b1)
-        h = norm2(x);   x += ffn(h) * sigmoid(R2 h + b2)
+        h = norm1(x);   x += m mixer(h + conv(h)) * sigmoid(R1 h + b1)
+        h = norm2(x);   x += m ffn(h) * sigmoid(R2 h + b2)
 
-    The gates read h as the norm left it, before the convolution. Options: ``taps`` (0: no convolution, the mixer reads h) with ``conv``
+    The gates read h as the norm left it, before the convolution. Options: ``residual_mult`` m (default 1); ``taps`` (0: no convolution, the mixer reads h) with ``conv``
     the name of its weights [size, taps]; ``gates``: the names of R1 and R2 [size, size], whose biases have ``bias_suffix`` added (None:
     no gates). A mixer whose output projection has a bias (``out_bias``) leaves it to the kernel that updates the stream; a
     routed feed-forward leaves a token's rows apart for it. The norms are of a kind that offers ``gated_add`` (``rmsnorm32``)."""
@@ -273,6 +274,7 @@ class GatedBlock(Part):
         self.mixer, self.feed_forward = mixer, feed_forward
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
         o = spec.options
+        self.mult = float(o.get("residual_mult", 1.0))
         self.taps = int(o.get("taps") or 0)
         # Kept [taps, size]: neighbouring channels' weights of one tap lie together.
         self.conv = rt.param(tensors[o["conv"]]).t().contiguous() if self.taps else None
@@ -315,9 +317,9 @@ class GatedBlock(Part):
         delta = self.mixer.forward(self.rt.buffer(ConvolvedRead.OUT, tuple(h.shape)) if self.taps else h, step, cache)
         bias = getattr(self.mixer, "out_bias", None)
         if self.feed_forward is None:
-            next_norm.gated_add(x, delta, h_out, bias=bias, **gate)
+            next_norm.gated_add(x, delta, h_out, bias=bias, mult=self.mult, **gate)
             return h_out
-        self.feed_forward_norm.gated_add(x, delta, h, bias=bias, **gate)
+        self.feed_forward_norm.gated_add(x, delta, h, bias=bias, mult=self.mult, **gate)
         gate = self._gate(1, h)
-        next_norm.gated_add(x, self.feed_forward.forward(h, step), h_out, **gate)
+        next_norm.gated_add(x, self.feed_forward.forward(h, step), h_out, mult=self.mult, **gate)
         return h_out

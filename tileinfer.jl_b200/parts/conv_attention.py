@@ -30,13 +30,16 @@ logarithmic steps up to ``far``, the last row from there on. In bfloat16 attenti
 library's paged kernels (tensor-memory and ``mma.sync`` prompt kernels, split-KV decode kernel; the bias comes as a table by distance),
 in 32-bit in the plain kernel.
 
+``norm_last``: the heads' norms come after the rotation instead of before it. ``keep_first``: beside the window, the sequence's first
+positions stay visible (at their true positions). ``sink`` "zero": the sink's score is 0 for every head, a one in the denominator.
+
 ``shared_kv``: there is no value projection; a token's values are its keys as projected (bias and convolution included), before norm and
 rotation. ``softcap`` c: the scaled score s becomes c tanh(s / c) before any bias. ``slopes`` (one number per head): slope * (i - j) is
 taken off the score after the cap, a linear bias by distance. Both run in every paged kernel.
 
 Record: ``num_heads``, ``num_kv_heads``, ``head_dim``, ``scale``, ``window``, ``kv_source``, ``qk_norm_eps`` and the options
 ``value_dim``, ``conv_taps`` (0: none), ``bias``, ``out_bias``, ``row_norm``, ``head_norm``, ``norm_weight``, ``sink``, ``gate``,
-``chunk``, ``distance_bias``, ``shared_kv``, ``softcap``, ``slopes``.
+``chunk``, ``distance_bias``, ``shared_kv``, ``softcap``, ``slopes``, ``norm_last``, ``keep_first``.
 """
 from __future__ import annotations
 
@@ -125,7 +128,13 @@ class ConvAttention(Mixer):
             self.slopes = exact.float().to(rt.device)
             self.slopes2 = (exact * 1.4426950408889634).float().to(rt.device)          # for the kernels that work in base 2
         self.out_name, self.gated_name = "mixer.delta", "conv_attention.gated"
-        self.sink = rt.param(tensors[p + n["sink"]], keep_dtype=True).float().contiguous() if self.sink_on else None
+        self.norm_last, self.keep = bool(o.get("norm_last", False)), int(o.get("keep_first") or 0)
+        if self.norm_last and not (self.row_norm and self.head_norm):
+            raise ValueError("conv_attention: a norm after the rotation is one of every head by itself")
+        if o.get("sink") == "zero":
+            self.sink = torch.zeros(self.nq, dtype=torch.float32, device=rt.device)
+        else:
+            self.sink = rt.param(tensors[p + n["sink"]], keep_dtype=True).float().contiguous() if self.sink_on else None
         self.o = Linear(get(n["o"]), rt, "o")
         self.o.partials_name = "mixer.partials"
         self.rotation = position.rotation() if position is not None else None
@@ -153,7 +162,7 @@ class ConvAttention(Mixer):
                 out.append(TensorDecl(p + n[k] + n["conv_suffix"], (r, taps), ("const_plus_normal", 1.0 / taps, 0.3)))
             if row_norm and k != "v" and o.get("norm_weight", True):
                 out.append(TensorDecl(p + n[k] + n["norm_suffix"], (D if o.get("head_norm", False) else r,), ("one_plus_normal", 0.1)))
-        if sink:
+        if sink and o.get("sink") != "zero":
             out.append(TensorDecl(p + n["sink"], (H,), ("normal", 1.0), keep_dtype=True))
         if gate:
             out.append(TensorDecl(p + n["g"], (H if o.get("gate") == "head" else H * V, W), std(W)))
@@ -164,7 +173,7 @@ class ConvAttention(Mixer):
     def cache_request(self):
         out = []
         if self.own_kv:
-            out.append(CacheRequest("paged_kv", kv_heads=self.nkv, head_dim=self.padded, window=self.spec.window))
+            out.append(CacheRequest("paged_kv", kv_heads=self.nkv, head_dim=self.padded, window=self.spec.window, keep_first=self.keep))
         if self.taps > 1:
             out.append(CacheRequest("state", shape=(self.taps - 1, self.channels), dtype=torch.float32))
         return tuple(out)
@@ -185,7 +194,7 @@ class ConvAttention(Mixer):
         meta = step.group(cache.group_index)
         ops.conv_attention_inputs(rows, self.bias, self.conv, self.taps, cache.state, self.q_norm, self.k_norm, s.qk_norm_eps, self.rotation,
                                   q, cache.k, cache.v, step, meta.slot_mapping, nq, nkv, D, V, Dp, cache.page_size, write_kv=self.own_kv,
-                                  head_norm=self.head_norm, shared_kv=self.shared_kv)
+                                  head_norm=self.head_norm, shared_kv=self.shared_kv, norm_last=self.norm_last)
         if self.taps > 1:
             ops.conv_state_update(cache.state, rows, self.bias, self.taps, step, C)
         attn = rt.buffer("attention.out", (n, nq * Dp))
@@ -193,11 +202,11 @@ class ConvAttention(Mixer):
         if rt.fast:
             from ..kernels import fast
             done = fast.attention(attn, q, cache, meta, step, self.attn_spec, sink=self.sink, chunk=self.chunk, distance_bias2=self.distance_bias2,
-                                  cap=self.softcap, slopes2=self.slopes2)
+                                  cap=self.softcap, slopes2=self.slopes2, keep=self.keep)
         if not done:
             ops.attention_plain(attn, q, cache.k, cache.v, meta.block_table, step.tok_slot, step.positions, s.scale, nq, nkv, Dp,
                                 cache.page_size, window=s.window or 0, sink=self.sink, chunk=self.chunk, distance_bias=self.distance_bias,
-                                cap=self.softcap, slopes=self.slopes)
+                                cap=self.softcap, slopes=self.slopes, keep=self.keep)
         if self.gated or Dp != V:
             y = rt.buffer(self.gated_name, (n, nq * V))
             ops.sigmoid_gate(y, attn, rows[:, C:] if self.gated else None, nq, V, Dp, per_head=self.gate_per_head)

@@ -22,10 +22,13 @@ Optional parts, by the record's options:
   (Wuk_h^T and an identity block) does both. The attended row's first kv_rank elements are the attended latent; Wuv_h is
   stored with zero columns behind them.
 * ``sink``: a learned number per head whose exponential is one more term of the softmax's denominator.
+* ``q_rank`` 0: there is no query latent, q_h = Wq_h h (tensor name ``q``).
+* ``keep_first``: beside the window, the sequence's first positions stay visible.
 * ``gate``: the heads' outputs are multiplied by sigmoid(Wg h) before Wo; Wg rides along in the down projection.
 
 Sizes and constants come from the record: ``num_heads``, ``head_dim`` (unrotated query/key size), ``scale``, ``window`` and the
-options ``value_dim``, ``q_rank``, ``kv_rank``, ``latent_norm_eps``, ``rot_dim``, ``sink``, ``gate``.
+options ``value_dim``, ``q_rank``, ``kv_rank``, ``latent_norm_eps``, ``rot_dim``, ``sink``, ``gate``,
+``keep_first``.
 """
 from __future__ import annotations
 
@@ -69,10 +72,13 @@ class LatentAttention(Mixer):
             raise ValueError(f"latent_attention: a cached row of {self.kv_rank} + {self.rot_dim} exceeds the attention kernels' {ops.MAX_HEAD_DIM}")
         n, p = spec.tensor_names, spec.prefix
         get = lambda k: rt.param(tensors[p + n[k]])
+        self.keep = int(o.get("keep_first") or 0)
         # The down projections (and the gate's) read the same input: one product, query latent first.
-        self.down = Linear(torch.cat([get("dq"), get("dkv")] + ([get("g")] if self.gated else []), 0).contiguous(), rt, "latent_down")
-        self.w_q_norm, self.w_kv_norm = get("dq_norm"), get("dkv_norm")
-        self.uq = Linear(get("uq"), rt, "uq")
+        down = ([get("dq")] if self.q_rank else []) + [get("dkv")] + ([get("g")] if self.gated else [])
+        self.down = Linear(torch.cat(down, 0).contiguous(), rt, "latent_down")
+        self.w_q_norm, self.w_kv_norm = get("dq_norm") if self.q_rank else None, get("dkv_norm")
+        # Queries from their latent, or straight from the mixer's input.
+        self.uq = Linear(get("uq" if self.q_rank else "q"), rt, "uq")
         H, D, V, R, Rd, P = self.heads, self.dim, self.vdim, self.kv_rank, self.rot_dim, self.pool_row
         # Wuk_h [dim, kv_rank] is used transposed (query -> the cached row's space); stored so, head after head, with an
         # identity block that passes the query's rotated part through and zero rows up to the cached row's length.
@@ -98,10 +104,14 @@ class LatentAttention(Mixer):
         W, H, D, V = spec.hidden_size, spec.num_heads, spec.head_dim, int(o["value_dim"])
         Q, R, Rd = int(o["q_rank"]), int(o["kv_rank"]), int(o.get("rot_dim", 0))
         std = lambda fan_in: ("normal", fan_in ** -0.5)
-        out = [TensorDecl(p + n["dq"], (Q, W), std(W)), TensorDecl(p + n["dq_norm"], (Q,), ("one_plus_normal", 0.1)),
-               TensorDecl(p + n["uq"], (H * (D + Rd), Q), std(Q)), TensorDecl(p + n["dkv"], (R + Rd, W), std(W)),
-               TensorDecl(p + n["dkv_norm"], (R,), ("one_plus_normal", 0.1)), TensorDecl(p + n["uk"], (H * D, R), std(R)),
-               TensorDecl(p + n["uv"], (H * V, R), std(R)), TensorDecl(p + n["o"], (W, H * V), std(H * V))]
+        if Q:
+            out = [TensorDecl(p + n["dq"], (Q, W), std(W)), TensorDecl(p + n["dq_norm"], (Q,), ("one_plus_normal", 0.1)),
+                   TensorDecl(p + n["uq"], (H * (D + Rd), Q), std(Q))]
+        else:
+            out = [TensorDecl(p + n["q"], (H * (D + Rd), W), std(W))]
+        out += [TensorDecl(p + n["dkv"], (R + Rd, W), std(W)),
+                TensorDecl(p + n["dkv_norm"], (R,), ("one_plus_normal", 0.1)), TensorDecl(p + n["uk"], (H * D, R), std(R)),
+                TensorDecl(p + n["uv"], (H * V, R), std(R)), TensorDecl(p + n["o"], (W, H * V), std(H * V))]
         if o.get("sink", False):
             out.append(TensorDecl(p + n["sink"], (H,), ("normal", 1.0), keep_dtype=True))
         if o.get("gate", False):
@@ -109,7 +119,7 @@ class LatentAttention(Mixer):
         return out
 
     def cache_request(self):
-        return CacheRequest("paged_latent", kv_heads=1, head_dim=self.pool_row, window=self.spec.window)
+        return CacheRequest("paged_latent", kv_heads=1, head_dim=self.pool_row, window=self.spec.window, keep_first=self.keep)
 
     def decode_plan(self, group):
         if not (self.rt.fast and self.rt.dtype == torch.bfloat16):
@@ -124,12 +134,12 @@ class LatentAttention(Mixer):
         rows = rt.buffer("latent.down", (n, self.down.out_features))
         # The gate's columns are read as they are by the gate's kernel: only a product without them may come in partial sums.
         rows = self.down.forward(h, rows, allow_partials=n <= 256 and not self.gated)
-        cq = rt.buffer("latent.cq", (n, Q))
+        cq = rt.buffer("latent.cq", (n, Q)) if Q else None
         meta = step.group(cache.group_index)
         ops.latent_inputs(rows, cq, cache.k, self.w_q_norm, self.w_kv_norm, self.eps, meta.slot_mapping, Q, R, self.rotation,
                           step.positions, P)
         q = rt.buffer("latent.q", (n, H, D + Rd))
-        self.uq.forward(cq, q.view(n, H * (D + Rd)))
+        self.uq.forward(cq if Q else h, q.view(n, H * (D + Rd)))
         if Rd:
             ops.rotate_heads(q, self.rotation, step.positions, first=D)
         fast = None
@@ -141,10 +151,10 @@ class LatentAttention(Mixer):
         attn = rt.buffer("latent.attended", (n, H, P))
         done = False
         if fast is not None:
-            done = fast.attention(attn.view(n, H * P), q_lat, cache, meta, step, self.attn_spec, sink=self.sink)
+            done = fast.attention(attn.view(n, H * P), q_lat, cache, meta, step, self.attn_spec, sink=self.sink, keep=self.keep)
         if not done:
             ops.attention_plain(attn.view(n, H * P), q_lat, cache.k, cache.v, meta.block_table, step.tok_slot, step.positions,
-                                s.scale, H, 1, P, cache.page_size, window=s.window or 0, sink=self.sink)
+                                s.scale, H, 1, P, cache.page_size, window=s.window or 0, sink=self.sink, keep=self.keep)
         values = rt.buffer("latent.values", (n, H, V))
         if not (fast is not None and fast.head_linear(values, attn, self.uv)):
             ops.head_gemm(values, attn, self.uv)

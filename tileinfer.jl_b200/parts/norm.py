@@ -68,16 +68,17 @@ class RMSNorm32(Norm):
         self._one_group("as the next norm of branch_add")
         return (self.weight, self.eps, self.offset)
 
-    def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None, conv=None):
-        """x += (delta + bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``delta`` None: x stays), then out = norm(x). ``delta``:
+    def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None, conv=None, mult=1.0):
+        """x += mult * (delta + bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``delta`` None: x stays), then out = norm(x). ``delta``:
         rows, 32-bit partial sums or :class:`GatheredRows` with weights; ``gate``: rows or partial sums, None for no gate. ``conv``: see
         ``ops.gated_add_norm32``."""
-        if self.offset:
-            raise NotImplementedError("a gain stored minus one, or a mean taken off, is not built for gated_add")
+        if self.offset not in (False, True):
+            raise NotImplementedError("a mean taken off is not built for gated_add")
+        common = dict(conv=conv, mult=mult, offset=self.offset)
         if isinstance(delta, GatheredRows):
-            ops.gated_add_norm32(x, delta.rows, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, delta.index, delta.scores, conv)
+            ops.gated_add_norm32(x, delta.rows, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, delta.index, delta.scores, **common)
         else:
-            ops.gated_add_norm32(x, delta, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, conv=conv)
+            ops.gated_add_norm32(x, delta, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, **common)
         return out
 
     def forward(self, x, out):

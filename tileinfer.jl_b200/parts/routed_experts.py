@@ -14,6 +14,8 @@ Options of the record: ``experts``, ``top``, ``limit`` (None: no clamp), ``sigmo
 (any of the following options) is chosen by ``csrc/routed_experts.cu``'s ``router_select``:
 
     ``score`` "softmax": s = softmax(z) over all router outputs instead of sigmoid(z)
+    ``score`` "chosen": the choice is by z itself and the weights are the softmax over the chosen logits alone
+    ``logit_bias``: a tensor added to z before anything else
     ``correction``: a tensor added to s for the CHOICE only (the weights use s)
     ``groups`` (count, keep): the router's outputs form `count` equal groups of neighbours, a group's score is its largest choice
         score, or with ``group_best`` 2 the sum of its two largest, and only members of the `keep` best groups can be chosen
@@ -42,7 +44,7 @@ from .norm import GatheredRows
 
 def _has_rules(o) -> bool:
     return bool(o.get("score", "sigmoid") != "sigmoid" or o.get("renormalize") or o.get("groups") or o.get("pass_through")
-                or o.get("correction") or o.get("shared_gate"))
+                or o.get("correction") or o.get("shared_gate") or o.get("logit_bias"))
 
 
 @register_feed_forward("routed_experts")
@@ -60,19 +62,25 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: a unit without a gate has the activation relu2, no clamp and no shared unit")
         self.select = _has_rules(o)
         self.softmax, self.renormalize = o.get("score", "sigmoid") == "softmax", bool(o.get("renormalize", False))
+        self.on_logits = o.get("score") == "chosen"
+        if self.on_logits:
+            self.renormalize = True
+            if o.get("correction") or (o.get("groups") and o["groups"][0] != o["groups"][1]):
+                raise ValueError("routed_experts: a choice on the logits has no correction and no groups")
         self.pass_through = int(o.get("pass_through", 0))
         self.groups, self.keep = (int(v) for v in (o.get("groups") or (1, 1)))
         self.group_best = int(o.get("group_best", 1))
         # Set by a block whose stream update adds up a token's rows itself: the output then comes as GatheredRows with their weights.
         self.rows_apart = False
-        if o.get("score", "sigmoid") not in ("sigmoid", "softmax"):
-            raise ValueError(f"routed_experts: score {o.get('score')!r} (known: sigmoid, softmax)")
+        if o.get("score", "sigmoid") not in ("sigmoid", "softmax", "chosen"):
+            raise ValueError(f"routed_experts: score {o.get('score')!r} (known: sigmoid, softmax, chosen)")
         if self.select and self.scale_input:
             raise ValueError("routed_experts: a router with rules scales the experts' outputs, not their inputs")
         total = self.experts + self.pass_through
         if total % self.groups or not 1 <= self.keep <= self.groups or self.keep * (total // self.groups) < self.top:
             raise ValueError(f"routed_experts: {self.keep} of {self.groups} groups over {total} router outputs for top {self.top}")
         self.correction = rt.param(tensors[p + n["correction"]], keep_dtype=True).float().contiguous() if o.get("correction") else None
+        self.logit_bias = rt.param(tensors[p + n["logit_bias"]], keep_dtype=True).float().contiguous() if o.get("logit_bias") else None
         self.gate_on = bool(o.get("shared_gate")) and int(o.get("shared_size", 0)) > 0
         self.router = get(n["router"])
         if self.gate_on:                         # the gate's row rides along as the router product's last output
@@ -115,6 +123,8 @@ class RoutedExperts(FeedForward):
         std = lambda fan_in: ("normal", fan_in ** -0.5)
         total = int(o["experts"]) + int(o.get("pass_through", 0))
         out = [TensorDecl(p + n["router"], (total, W), std(W))]
+        if o.get("logit_bias"):
+            out.append(TensorDecl(p + n["logit_bias"], (total,), ("normal", 0.1), keep_dtype=True))
         if o.get("correction"):
             out.append(TensorDecl(p + n["correction"], (total,), ("normal", 0.02), keep_dtype=True))
         if o.get("shared_gate") and int(o.get("shared_size", 0)):
@@ -153,7 +163,7 @@ class RoutedExperts(FeedForward):
             pass_weight = rt.buffer("experts.pass_weight", (n,), torch.float32) if self.pass_through else None
             ops.router_select(h, self.router, logits, E, E + self.pass_through, top, ids, scores, pass_weight, softmax=self.softmax,
                               correction=self.correction, groups=self.groups, keep=self.keep, group_best=self.group_best, renormalize=self.renormalize,
-                              always=self.always, gate=self.gate_on)
+                              always=self.always, gate=self.gate_on, logit_bias=self.logit_bias, on_logits=self.on_logits)
         else:
             ops.router_topk(h, self.router, top, ids, scores, logits, always=self.always)
         ops.expert_plan(ids, self.units, tile, pair_row, row_pair, plan)
