@@ -9,6 +9,7 @@ model with random weights (bfloat16), plus prefill throughput and roofline fract
     python bench.py --preset sozanex [--timeline]  (the Sozanex design at two sizes beside Vogilix layers of equal size)
     python bench.py --preset fasodra [--timeline]  (the Fasodra design at two sizes beside Zudepel layers of equal size)
     python bench.py --preset midisun [--timeline]  (the Midisun design at two sizes beside Zudepel layers of equal size)
+    python bench.py --preset pemarax [--timeline]  (the Pemarax design at two sizes beside Fasodra layers of equal size)
 
 Prints one JSON line. A "step" is one decode step of the whole batch (default batch 8, every
 sequence after 1,023 cached positions, context 4,096). ``value`` is decoded tokens per second
@@ -652,6 +653,31 @@ def midisun_config(size: str, layers: int):
             "layers": [{"mixer": m, "mlp": {"ff": dense, "kind": "dense"} if i == 0 else moe, "type": t} for i, (t, m) in enumerate(kinds)]}
 
 
+def pemarax_config(size: str, layers: int):
+    """Layers of a real model's sizes: attention beside a state-space recurrence of twice the width, windowed attention with kept first
+    positions behind short convolutions, and two layers of latent attention, in turn; every layer with routed squared-rectifier experts."""
+    w, heads, kv_heads, dim, experts, top, ff, vocab, window, latent, groups = {
+        "mid": (2048, 16, 4, 128, 32, 4, 1024, 32768, 1024, (64, 32, 96), 1),
+        "wide": (4096, 32, 8, 128, 64, 6, 1408, 65536, 2048, (128, 64, 192), 8)}[size]
+    moe = {"expert": {"ff": ff}, "kind": "moe", "router": {"experts": experts, "top": top}}
+    grouped = {"dim": dim, "heads": heads, "kv_heads": kv_heads, "scale": dim ** -0.5, "vdim": dim}
+    yarn = {"factor": 4.0, "fast": 32.0, "original": 4096, "slow": 1.0}
+    ldim, rot, rank = latent
+    mixers = [("parallel", {"left": {**grouped, "mask": {"size": window}},
+                            "right": {"conv": 4, "groups": groups, "heads": 2 * w // 64, "norm_groups": groups, "state": 128, "vdim": 64}}),
+              ("attention", {**grouped, "conv": 4, "mask": {"keep_first": 64, "size": window}, "rot": {"base": 500000.0, "dims": dim, "scaling": yarn}}),
+              ("latent_attention", {"dim": ldim, "heads": heads, "kv_rank": rank, "mask": {"size": window}, "rot": {"base": 10000.0, "dims": rot}, "rot_dim": rot,
+                                    "scale": (ldim + rot) ** -0.5, "vdim": ldim})]
+    kinds = [mixers[(0, 1, 2, 2)[i % 4]] for i in range(layers)]
+    return {"architecture": "Pemarax", "vocab": vocab, "width": w, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "layers": [{"mixer": m, "mlp": moe, "type": t} for t, m in kinds]}
+
+
+def fasodra_twin(size: str, layers: int):
+    """Fasodra layers beside a Pemarax configuration: the same width, depth, heads, experts and expert size, one copy of the stream."""
+    return {**fasodra_config(size, layers), "streams": 0}
+
+
 def run_beside(args, pk_source, name, config, twin, twin_config):
     """Prefill and decode throughput of a design at two sizes, each beside layers of another of the library's designs of the same width,
     depth, heads, experts and expert sizes; with --timeline also the per-kernel device times of one prompt step and one decode step of
@@ -733,7 +759,7 @@ def main(argv=None) -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (quick checks)")
     ap.add_argument("--timeline", action="store_true", help="--preset vogilix: per-kernel device times of its steps, on stderr")
-    ap.add_argument("--preset", default="8b", choices=["8b", "8b-long", "70b", "sweep", "vogilix", "zudepel", "sozanex", "fasodra", "midisun"],
+    ap.add_argument("--preset", default="8b", choices=["8b", "8b-long", "70b", "sweep", "vogilix", "zudepel", "sozanex", "fasodra", "midisun", "pemarax"],
                     help="8b: the headline line (default); 8b-long: 8 unequal sequences of up to 32,768 positions; "
                          "70b: Apertus-70B sizes, 141 GB of weights")
     args = ap.parse_args(argv)
@@ -763,6 +789,8 @@ def main(argv=None) -> int:
         return run_beside(args, peaks()[1], "fasodra", fasodra_config, "zudepel", zudepel_config)
     if args.preset == "midisun":
         return run_beside(args, peaks()[1], "midisun", midisun_config, "zudepel", zudepel_config)
+    if args.preset == "pemarax":
+        return run_beside(args, peaks()[1], "pemarax", pemarax_config, "fasodra", fasodra_twin)
     if args.preset == "sozanex":
         return run_sozanex(args, *peaks())
     if args.preset == "zudepel":

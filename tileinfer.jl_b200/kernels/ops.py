@@ -476,8 +476,6 @@ def expert_combine(out, y, pair_row, scores, shared, top, scale_output=False, h=
     _need(out, "out"); _need(y, "y", out.dtype); _need(pair_row, "pair_row", torch.int32); _need(scores, "scores", torch.float32)
     if shared is not None:
         _need(shared, "shared", out.dtype)
-    if logit_bias is not None:
-        _need(logit_bias, "logit_bias", torch.float32)
     if pass_weight is not None:
         _need(pass_weight, "pass_weight", torch.float32); _need(h, "h", out.dtype)
     n, width = out.shape

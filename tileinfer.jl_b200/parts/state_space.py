@@ -23,6 +23,13 @@ from .base import CacheRequest, Mixer, register_mixer
 from .linear import Linear
 
 
+def chunk_step(rt, y, xbc, coef, skip, state, step, heads, groups, dim, vdim):
+    """The recurrence over a step of several tokens per sequence, with its work space from the runtime's scratch buffers."""
+    chunks, floats = ops.memory_chunk_sizes(step.host_q_lens, heads, dim, vdim)
+    ws, total = rt.buffer("memory.chunks", (floats,), torch.float32), rt.buffer("memory.totals", (chunks, heads), torch.float32)
+    ops.ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, total, chunks)
+
+
 @register_mixer("state_space")
 class StateSpace(Mixer):
     def __init__(self, spec: MixerSpec, tensors, rt, position):
@@ -80,9 +87,7 @@ class StateSpace(Mixer):
         else:
             if self.taps > 1:
                 ops.history_update(hist, rows[:, self.inner:], self.taps, step, self.channels)
-            chunks, floats = ops.memory_chunk_sizes(step.host_q_lens, self.heads, self.dim, self.vdim)
-            ws, total = rt.buffer("memory.chunks", (floats,), torch.float32), rt.buffer("memory.totals", (chunks, self.heads), torch.float32)
-            ops.ssm_chunks(y, xbc, coef, self.skip, state, step, *sizes, ws, total, chunks)
+            chunk_step(rt, y, xbc, coef, self.skip, state, step, *sizes)
         gated = rt.buffer("state_space.normed", (n, self.inner))
         ops.ssm_gate_norm(gated, y, rows[:, :self.inner], self.norm_w, self.eps, self.parts)
         return self.o.forward(gated, rt.buffer(self.out_name, (n, self.spec.hidden_size)), allow_partials=True)
