@@ -19,10 +19,10 @@
 //
 // q and k are rotated by the token's position and scaled while they are staged, in 32-bit. L is summed in 64-bit: a difference of two
 // large sums must not lose the small decay between neighbours.
-#include "common.cuh"
+#include "chunk_index.cuh"
 #include "mma_util.cuh"
 
-#define MC_TOKENS 64
+#define MC_TOKENS CHUNK_TOKENS
 #define MC_SLAB 128              // key rows and value columns staged at once
 #define MC_PITCH (MC_SLAB + 4)   // floats between staged rows: eight rows' 16-byte pieces lie in different banks
 #define MC_THREADS 256
@@ -49,32 +49,6 @@ struct ChunkArgs {
     long long ws_pitch;
     float* total;                // [chunks, H]: e^(L_64)
 };
-
-// The tokens of chunk `c` of the step: false beyond the last one. Every warp looks at 32 sequences at once.
-__device__ __forceinline__ bool chunk_of(const ChunkArgs& a, int c, int& t0, int& count) {
-    const int lane = threadIdx.x & 31;
-    for (int b0 = 0; b0 < a.B; b0 += 32) {
-        const int b = b0 + lane;
-        const int lo = b < a.B ? __ldcg(a.cu_seqlens + b) : 0, len = b < a.B ? __ldcg(a.cu_seqlens + b + 1) - lo : 0;
-        const int chunks = (len + MC_TOKENS - 1) / MC_TOKENS;
-        int upto = chunks;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const int p = __shfl_up_sync(0xffffffffu, upto, o);
-            if (lane >= o) upto += p;
-        }
-        const unsigned after = __ballot_sync(0xffffffffu, c < upto);
-        if (after != 0) {
-            const int owner = __ffs(after) - 1;
-            const int k = c - __shfl_sync(0xffffffffu, upto - chunks, owner);
-            t0 = __shfl_sync(0xffffffffu, lo, owner) + k * MC_TOKENS;
-            count = min(MC_TOKENS, __shfl_sync(0xffffffffu, len, owner) - k * MC_TOKENS);
-            return true;
-        }
-        c -= __shfl_sync(0xffffffffu, upto, 31);
-    }
-    return false;
-}
 
 // L and b of the chunk's tokens (beyond `count`: L stays, b is zero). 64 threads; the caller synchronises.
 __device__ __forceinline__ void chunk_decays(const ChunkArgs& a, int h, int t0, int count, double* L, float* add) {
@@ -199,7 +173,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_states_kernel(Chun
     const int d0 = (blockIdx.z / v_slabs) * MC_SLAB, v0 = (blockIdx.z % v_slabs) * MC_SLAB;
     int t0 = 0, count = 0;
     pdl_enter();
-    if (!chunk_of(a, blockIdx.x, t0, count)) return;
+    if (!chunk_of(a.cu_seqlens, a.B, blockIdx.x, t0, count)) return;
     chunk_decays(a, h, t0, count, L, add);
     __syncthreads();
     chunk_join(L);
@@ -255,10 +229,7 @@ __global__ void __launch_bounds__(256) memory_chunk_scan_kernel(ChunkArgs a, flo
     const int DV = a.D * a.V, elements = DV + (a.vector ? a.D : 0);
     const int e = (blockIdx.x * 256 + threadIdx.x) * VEC;
     pdl_enter();
-    int first = 0;                                       // chunks of the sequences before this one: a warp counts 32 sequences at once
-    for (int i = threadIdx.x & 31; i < b; i += 32) first += (__ldcg(a.cu_seqlens + i + 1) - __ldcg(a.cu_seqlens + i) + MC_TOKENS - 1) / MC_TOKENS;
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) first += __shfl_xor_sync(0xffffffffu, first, o);
+    const int first = chunks_before(a.cu_seqlens, b);
     const int chunks = (__ldcg(a.cu_seqlens + b + 1) - __ldcg(a.cu_seqlens + b) + MC_TOKENS - 1) / MC_TOKENS;
     if (e >= elements) return;
     float* base = state + (size_t)__ldcg(seq_slots + b) * state_stride;
@@ -321,7 +292,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunk_outputs_kernel(Chu
     const bool gated = a.vector != 0;
     int t0 = 0, count = 0;
     pdl_enter();
-    if (!chunk_of(a, blockIdx.x, t0, count)) return;
+    if (!chunk_of(a.cu_seqlens, a.B, blockIdx.x, t0, count)) return;
     chunk_decays(a, h, t0, count, L, add);
     __syncthreads();
     chunk_join(L);

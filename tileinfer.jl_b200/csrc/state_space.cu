@@ -13,7 +13,8 @@
 #include "common.cuh"
 
 #define SI_MAX_TAPS 16
-#define SI_TOKENS 16
+#define SI_TOKENS 16             // rows a block walks in steps of several tokens per sequence
+#define SI_AHEAD 4               // rows whose loads are in flight together
 
 __device__ __forceinline__ float ssm_silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float ssm_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
@@ -53,14 +54,14 @@ struct SsmInputs {
     const float* a_log;          // [H]
     const int* cu_seqlens;
     const int* seq_slots;
-    int B, n, decode;
+    int B, n, decode, tokens;    // tokens: rows of a block
 };
 
-// Blocks (channels, rows of SI_TOKENS tokens), and one more column of blocks for (l, dt). conv is [taps][C].
+// Blocks (channels, `tokens` rows), and one more column of blocks for (l, dt). conv is [taps][C].
 template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(128) ssm_inputs_kernel(T* __restrict__ xbc, float* __restrict__ coef, const T* rows, const T* __restrict__ conv,
                                                          const T* __restrict__ bias, SsmInputs a) {
-    const int first = blockIdx.y * SI_TOKENS, last = min(a.n, first + SI_TOKENS);
+    const int first = blockIdx.y * a.tokens, last = min(a.n, first + a.tokens);
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     const int ntaps = TAPS > 0 ? TAPS : a.taps;
     constexpr int SLOTS = TAPS > 0 ? TAPS : 1, BACK = TAPS > 1 ? TAPS - 1 : 1;
@@ -93,37 +94,60 @@ __global__ void __launch_bounds__(128) ssm_inputs_kernel(T* __restrict__ xbc, fl
         if (r >= begin) Cells<T, VEC>::load(src + (size_t)r * a.ld, u);
         else Cells<float, VEC>::load(a.hist + (size_t)__ldcg(a.seq_slots + b) * a.hist_stride + (size_t)(ntaps - 1 - (begin - r)) * a.C + i, u);
     };
-    bool fresh = true;                                   // the rows before the current one are not in registers
-    for (int t = first; t < last; ++t) {
-        while (t >= end) { ++b; begin = __ldcg(a.cu_seqlens + b); end = __ldcg(a.cu_seqlens + b + 1); fresh = true; }
-        float u[VEC], acc[VEC];
-        Cells<T, VEC>::load(src + (size_t)t * a.ld, u);
+    auto finish = [&](int t, float (&acc)[VEC]) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+        for (int e = 0; e < VEC; ++e) {
+            const float z = acc[e] + bc[e];              // (16-bit rows: the fast exponential and division are far below their rounding)
+            acc[e] = sizeof(T) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : ssm_silu(z);
+        }
+        Cells<T, VEC>::store(xbc + (size_t)t * a.C + i, acc);
+    };
+    bool fresh = true;                                   // the rows before the current one are not in registers
+    int t = first;
+    while (t < last) {
+        while (t >= end) { ++b; begin = __ldcg(a.cu_seqlens + b); end = __ldcg(a.cu_seqlens + b + 1); fresh = true; }
         if (TAPS > 0) {
+            const int rows_now = min(SI_AHEAD, min(last, end) - t);
+            float u[SI_AHEAD][VEC];
+#pragma unroll
+            for (int q = 0; q < SI_AHEAD; ++q)
+                if (q < rows_now) Cells<T, VEC>::load(src + (size_t)(t + q) * a.ld, u[q]);
             if (TAPS > 1 && fresh)
 #pragma unroll
                 for (int j = 0; j < BACK; ++j) earlier(t - BACK + j, w[j]);
             fresh = false;
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; ++j)
+            for (int q = 0; q < SI_AHEAD; ++q) {
+                if (q >= rows_now) break;
+                float acc[VEC];
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) acc[e] = fmaf(c[j][e], w[j][e], acc[e]);
+                for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) acc[e] = fmaf(c[SLOTS - 1][e], u[e], acc[e]);
-            if (a.decode && TAPS > 1) {                  // one token per sequence: these channels' history moves up by one row
-                float* st = a.hist + (size_t)__ldcg(a.seq_slots + b) * a.hist_stride + i;
+                for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-                for (int j = 0; j + 1 < BACK; ++j) Cells<float, VEC>::store(st + (size_t)j * a.C, w[j + 1]);
-                Cells<float, VEC>::store(st + (size_t)(BACK - 1) * a.C, u);
+                    for (int e = 0; e < VEC; ++e) acc[e] = fmaf(c[j][e], w[j][e], acc[e]);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) acc[e] = fmaf(c[SLOTS - 1][e], u[q][e], acc[e]);
+                if (a.decode && TAPS > 1) {              // one token per sequence: these channels' history moves up by one row
+                    float* st = a.hist + (size_t)__ldcg(a.seq_slots + b) * a.hist_stride + i;
+#pragma unroll
+                    for (int j = 0; j + 1 < BACK; ++j) Cells<float, VEC>::store(st + (size_t)j * a.C, w[j + 1]);
+                    Cells<float, VEC>::store(st + (size_t)(BACK - 1) * a.C, u[q]);
+                }
+#pragma unroll
+                for (int j = 0; j + 1 < BACK; ++j)
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) w[j][e] = w[j + 1][e];
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) w[BACK - 1][e] = u[q][e];
+                finish(t + q, acc);
             }
-#pragma unroll
-            for (int j = 0; j + 1 < BACK; ++j)
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) w[j][e] = w[j + 1][e];
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) w[BACK - 1][e] = u[e];
+            t += rows_now;
         } else {
+            float u[VEC], acc[VEC];
+            Cells<T, VEC>::load(src + (size_t)t * a.ld, u);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
             float* st = a.hist + (size_t)__ldcg(a.seq_slots + b) * a.hist_stride + i;
             for (int j = 0; j < ntaps; ++j) {
                 float v[VEC], cj[VEC];
@@ -133,10 +157,9 @@ __global__ void __launch_bounds__(128) ssm_inputs_kernel(T* __restrict__ xbc, fl
                 for (int e = 0; e < VEC; ++e) acc[e] = fmaf(cj[e], j + 1 < ntaps ? v[e] : u[e], acc[e]);
                 if (a.decode && j > 0) Cells<float, VEC>::store(st + (size_t)(j - 1) * a.C, j + 1 < ntaps ? v : u);
             }
+            finish(t, acc);
+            ++t;
         }
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] = ssm_silu(acc[e] + bc[e]);
-        Cells<T, VEC>::store(xbc + (size_t)t * a.C + i, acc);
     }
 }
 
@@ -147,7 +170,7 @@ extern "C" int ti_ssm_inputs(void* xbc, float* coef, const void* rows, long long
                              int n, int B, int C, int H, int decode, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
     TI_REQUIRE(taps >= 1 && taps <= SI_MAX_TAPS && (taps == 1 || hist != nullptr) && C > 0 && H > 0 && B > 0, "ssm_inputs: %d taps, %d channels, %d heads", taps, C, H);
-    const SsmInputs a = {ld, x_off, dt_off, C, H, taps, hist, hist_stride, dt_bias, a_log, cu_seqlens, seq_slots, B, n, decode};
+    const SsmInputs a = {ld, x_off, dt_off, C, H, taps, hist, hist_stride, dt_bias, a_log, cu_seqlens, seq_slots, B, n, decode, decode ? 1 : SI_TOKENS};
 #define SI_LAUNCH(V, TAPS) ti_launch(ssm_inputs_kernel<T, V, TAPS>, grid, dim3(128), 0, stream, (T*)xbc, coef, (const T*)rows, (const T*)conv, (const T*)bias, a)
 #define SI_TAPS(V)                        \
     switch (taps) {                       \
@@ -161,7 +184,7 @@ extern "C" int ti_ssm_inputs(void* xbc, float* coef, const void* rows, long long
         const uintptr_t mask = sizeof(T) == 2 ? 7 : 15;
         const bool vec = C % 4 == 0 && ld % 4 == 0 && x_off % 4 == 0 && hist_stride % 4 == 0 && aligned16(hist) &&
                          (((uintptr_t)xbc | (uintptr_t)rows | (uintptr_t)conv | (uintptr_t)bias) & mask) == 0;
-        const dim3 grid((vec ? C / 4 + 127 : C + 127) / 128 + 1, (n + SI_TOKENS - 1) / SI_TOKENS);
+        const dim3 grid((vec ? C / 4 + 127 : C + 127) / 128 + 1, (n + a.tokens - 1) / a.tokens);
         if (vec) { SI_TAPS(4) } else { SI_TAPS(1) }
     });
 #undef SI_TAPS

@@ -91,7 +91,7 @@ _SIGNATURES = {
 }
 
 
-_KERNELS_PER_CALL = {"ti_memory_chunks": 3, "ti_ssm_chunks": 3}
+_KERNELS_PER_CALL = {"ti_memory_chunks": 3, "ti_ssm_chunks": 3, "ti_ssm_chunks_tc": 3}
 
 
 def lib():
@@ -252,5 +252,6 @@ _SIGNATURES.update({
     "ti_ssm_inputs": [_P, _P, _P, _L, _I, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "ti_ssm_token": [_P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "ti_ssm_chunks": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "ti_ssm_chunks_tc": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     "ti_ssm_gate_norm": [_P, _P, _P, _L, _P, _F, _I, _I, _I, _I, _P],
 })

@@ -887,8 +887,9 @@ def ssm_token(y, xbc, coef, skip, state, step, heads, groups, dim, vdim):
                              step.n_seqs, xbc.shape[1], heads, groups, dim, vdim, dtype_code(xbc.dtype), _stream()), "ssm_token")
 
 
-def ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, total, chunks):
-    """The same over a step's tokens in chunks of CHUNK_TOKENS. ``ws``, ``total`` [chunks, heads]: float32 work space (``memory_chunk_sizes``)."""
+def ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, total, chunks, tensor_cores=True):
+    """The same over a step's tokens in chunks of CHUNK_TOKENS; bfloat16 rows of sizes that csrc/ssm_chunks.cu takes go through it, unless
+    ``tensor_cores`` is off. ``ws``, ``total`` [chunks, heads]: float32 work space (``memory_chunk_sizes``)."""
     _need(y, "y", torch.float32); _need(xbc, "xbc"); _need(coef, "coef", torch.float32); _need(skip, "skip", torch.float32)
     for t, name in ((state, "state"), (ws, "ws"), (total, "total")):
         _need(t, name, torch.float32, contiguous=False)
@@ -896,9 +897,15 @@ def ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, to
         raise KernelError(f"ssm_chunks: rows of {xbc.shape[1]}, states of {state.shape[1]} for {heads} heads of {dim} x {vdim} in {groups} groups")
     if ws.numel() < chunks * heads * int(lib().ti_memory_chunk_pitch(dim, vdim)) or total.numel() < chunks * heads:
         raise KernelError(f"ssm_chunks: work space of {ws.numel()} floats for {chunks} chunks")
-    check(lib().ti_ssm_chunks(y.data_ptr(), xbc.data_ptr(), xbc.shape[1], 0, heads * vdim, heads * vdim + groups * dim, state.data_ptr(), state.stride(0),
-                              coef.data_ptr(), skip.data_ptr(), ws.data_ptr(), total.data_ptr(), chunks, step.cu_seqlens.data_ptr(),
-                              step.seq_slots.data_ptr(), step.n_seqs, heads, groups, dim, vdim, dtype_code(xbc.dtype), _stream()), "ssm_chunks")
+    args = (y.data_ptr(), xbc.data_ptr(), xbc.shape[1], 0, heads * vdim, heads * vdim + groups * dim, state.data_ptr(), state.stride(0), coef.data_ptr(),
+            skip.data_ptr(), ws.data_ptr(), total.data_ptr(), chunks, step.cu_seqlens.data_ptr(), step.seq_slots.data_ptr(), step.n_seqs, heads, groups,
+            dim, vdim)
+    if tensor_cores and xbc.dtype == torch.bfloat16:
+        rc = lib().ti_ssm_chunks_tc(*args, _stream())
+        if rc != 2:
+            check(rc, "ssm_chunks_tc")
+            return
+    check(lib().ti_ssm_chunks(*args, dtype_code(xbc.dtype), _stream()), "ssm_chunks")
 
 
 def ssm_gate_norm(out, y, z, w, eps, parts):

@@ -8,7 +8,8 @@ short convolution.
     out = W_o ( norm over ``norm_groups`` equal parts of (y silu(z)) * w )
 
 A sequence keeps the matrices S and the last taps - 1 rows of x | B | C, one block of floats. One-token steps run in ``ssm_token``, others in
-chunks of tokens that are worked on side by side (``csrc/memory_chunks.cu``); the recurrence and all that enters it from dt' on is 32-bit in
+chunks of tokens that are worked on side by side (``csrc/ssm_chunks.cu`` on the tensor cores, ``csrc/memory_chunks.cu`` in 32-bit and for the
+sizes the other refuses); the recurrence and all that enters it from dt' on is 32-bit in
 every element type.
 
 Record: ``num_heads``, ``head_dim`` (the state's size) and the options ``value_dim``, ``groups``, ``conv_taps``, ``norm_groups``, ``norm_eps``.
@@ -27,7 +28,7 @@ def chunk_step(rt, y, xbc, coef, skip, state, step, heads, groups, dim, vdim):
     """The recurrence over a step of several tokens per sequence, with its work space from the runtime's scratch buffers."""
     chunks, floats = ops.memory_chunk_sizes(step.host_q_lens, heads, dim, vdim)
     ws, total = rt.buffer("memory.chunks", (floats,), torch.float32), rt.buffer("memory.totals", (chunks, heads), torch.float32)
-    ops.ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, total, chunks)
+    ops.ssm_chunks(y, xbc, coef, skip, state, step, heads, groups, dim, vdim, ws, total, chunks, tensor_cores=rt.fast)
 
 
 @register_mixer("state_space")
