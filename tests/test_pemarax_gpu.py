@@ -165,11 +165,13 @@ def test_other_arrangements_of_layers(dtype):
     one = 1 if T == torch.float32 else 5          # rows of very few values normed are little more than signs, which rounding to bfloat16 may turn
     cases = {
         "attention only": pc.model(50, 24, 1e-4, 0.3, [pc.attention(3, 1, 6, 5, 0.3, D4, window=1, keep=1, conv=5), pc.attention(2, 2, 16, None, 0.5, None, window=2, keep=130),
-                                                        pc.attention(4, 1, 12, 20, 0.4, pc.moe(8, 4, 4), window=65, keep=64, rot=(4, 9.0))]),
+                                                        pc.attention(4, 1, 12, 20, 0.4, pc.moe(8, 4, 4), window=65, keep=64, rot=(4, 9.0)),
+                                                        pc.attention(16, 4, 32, 48, 0.3, None, window=40, keep=9, conv=4, rot=(30, 9.0))]),
         "latent only": pc.model(71, 40, 1e-5, 1.3, [pc.latent(2, 4, 2, 3, 5, 0.5, 30.0, D4, window=1), pc.latent(1, 50, 14, 60, 90, 0.2, 50.0, None),
                                                      pc.latent(5, 16, 8, 1, 250, 0.1, 10.0, pc.moe(12, 1, 1), window=128)]),
         "parallel only": pc.model(33, 32, 1e-6, 0.6, [pc.parallel((2, 1, 6, 5, 0.4, 3), (3, one, 1, 1, 9, 1), D4), pc.parallel((1, 1, 40, 8, 0.2, 100), (1, 150, 140, 1, 2, 1), None),
-                                                       pc.parallel((3, 3, 8, 16, 0.3, None), (8, 16, 32, 8, 4, 8), pc.moe(12, 3, 3))]),
+                                                       pc.parallel((3, 3, 8, 16, 0.3, None), (8, 16, 32, 8, 4, 8), pc.moe(12, 3, 3)),
+                                                       pc.parallel((20, 5, 36, 16, 0.3, 30), (4, 8, 16, 2, 4, 1), None)]),
     }
     with tempfile.TemporaryDirectory() as tmp:
         for name, case in cases.items():
@@ -546,6 +548,32 @@ def test_the_stream_update_with_a_multiplier_and_a_gain_around_zero(dtype):
 
 
 @pytest.mark.parametrize("dtype", sorted(DTYPES))
+def test_the_stream_update_by_two_normed_sublayers(dtype):
+    """Both sides as rows and as partial sums, of very different sizes, against the formula and against the sum made by a kernel of its own."""
+    from tileinfer_b200.kernels import ops
+    from tileinfer_b200.parts import Runtime
+    from tileinfer_b200.parts.norm import PairRows
+    T = DTYPES[dtype]
+    g = torch.Generator().manual_seed(8)
+    for size in (60, 33, 1024, 5000):
+        x, w = torch.randn(5, size, generator=g).double(), rnd(0.3 * torch.randn(size, generator=g, dtype=F64), T)
+        wa, wb = rnd(torch.randn(size, generator=g, dtype=F64), T), rnd(torch.randn(size, generator=g, dtype=F64), T)
+        a, b, parts = rnd(50 * torch.randn(5, size, generator=g, dtype=F64), T), rnd(0.02 * torch.randn(5, size, generator=g, dtype=F64), T), torch.randn(3, 5, size, generator=g)
+        for left, right, lv, rv in ((a.to(T).cuda(), b.to(T).cuda(), a, b), (parts.cuda(), b.to(T).cuda(), parts.double().sum(0), b),
+                                    (b.to(T).cuda(), parts.cuda(), b, parts.double().sum(0))):
+            pair = 0.7 * plain.rms_divide(lv, 1e-4) * wa + 0.4 * plain.rms_divide(rv, 1e-4) * wb
+            ref = x + 0.6 * pair
+            want = plain.offset_norm(ref, w, 1e-5)
+            xd, h = x.float().cuda(), torch.full((5, size), float("nan"), dtype=T, device="cuda")
+            wad, wbd = wa.to(T).cuda(), wb.to(T).cuda()
+            ops.pair_add_norm32(xd, left, right, wad, wbd, 0.7, 0.4, 1e-4, 0.6, h, w.to(T).cuda(), 1e-5, offset=True)
+            assert float((xd.cpu().double() - ref).abs().max()) <= 1e-5 * max(1.0, float(ref.abs().max()))
+            assert float((h.cpu().double() - want).abs().max()) <= (1e-5 if T == torch.float32 else 2.0 ** -7) * float(want.abs().max())
+            apart = PairRows(left, right, wad, wbd, 1e-4, 0.7, 0.4).combined(Runtime(T))
+            assert float((apart[0].cpu().double() - pair).abs().max()) <= 1e-5 * max(1.0, float(pair.abs().max()))
+
+
+@pytest.mark.parametrize("dtype", sorted(DTYPES))
 def test_router_that_chooses_on_biased_logits(dtype):
     """Biases that decide the choice, logits so far apart that a softmax over all of them would be zero for most, equal logits (the smaller
     index first), one expert and all of them."""
@@ -594,9 +622,9 @@ def test_bfloat16_steps_take_the_fast_kernels(models):
     engine.check_health()
     assert prompt.get("ti_attention_prefill_tc_kept", 0) == 3 and token.get("ti_attention_decode_kept", 0) == 3, (prompt, token)
     assert prompt.get("ti_attention_prefill_tc", 0) == 3 and prompt.get("ti_attention_prefill", 0) == 1, prompt
-    assert prompt.get("ti_ssm_inputs", 0) == 2 and token.get("ti_ssm_token", 0) == 2, (prompt, token)
+    assert prompt.get("ti_ssm_inputs", 0) == 2 and prompt.get("ti_ssm_chunks_tc", 0) == 2 and "ti_ssm_chunks" not in prompt and token.get("ti_ssm_token", 0) == 2, (prompt, token)
     for used in (prompt, token):
-        assert used.get("ti_gemm_tcgen05_grouped", 0) == 12 and used.get("ti_gated_add_norm32", 0) == 13, used
+        assert used.get("ti_gemm_tcgen05_grouped", 0) == 12 and used.get("ti_gated_add_norm32", 0) == 11 and used.get("ti_pair_add_norm32", 0) == 2, used
         assert not any(k.startswith(("ti_attention_plain", "ti_grouped_gemm", "ti_gemm_plain", "ti_expert_combine", "ti_head_gemm")) for k in used), used
     assert prompt.get("ti_gemm_tcgen05", 0) > 0 and token.get("ti_gemv_bf16", 0) > 0
 

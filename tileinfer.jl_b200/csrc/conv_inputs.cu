@@ -12,7 +12,9 @@
 // The last taps - 1 rows u of every sequence are its convolution state [slots][taps - 1][channels] (32-bit copies of the
 // T values, so a row read from the state equals the row read from the step's own projection bit for bit); tokens at the
 // start of a step read it, and `conv_state_update` (a second launch: the first one's blocks read what it overwrites)
-// moves it on. One block per token; everything between the loads and the one rounding per stage is 32-bit.
+// moves it on. One block per token, or, where no sum
+// runs over a whole row and a step has few tokens, several that share out its heads; everything between the loads and the one rounding per
+// stage is 32-bit.
 #include "common.cuh"
 
 #define CI_THREADS 256
@@ -39,6 +41,11 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
     __shared__ float scratch[33];
     const int t = blockIdx.x;
     const int Cq = nq * D, Ck = write_kv ? nkv * D : 0, Cv = write_kv && !shared_kv ? nkv * V : 0, C = Cq + Ck + Cv;
+    // This block's heads (queries, then keys, then values) and their channels.
+    const int qk = nq + (Ck > 0 ? nkv : 0), units = qk + (Cv > 0 ? nkv : 0);
+    const int u0 = units * (int)blockIdx.y / (int)gridDim.y, u1 = units * ((int)blockIdx.y + 1) / (int)gridDim.y;
+    auto channel = [&](int u) { return u <= qk ? u * D : qk * D + (u - qk) * V; };
+    const int c0 = channel(u0), c1 = channel(u1), qk0 = min(u0, qk), qk1 = min(u1, qk), v0 = max(u0 - qk, 0), v1 = max(u1 - qk, 0);
     const int p = __ldcg(positions + t);
     const int b = sequence_of(cu_seqlens, B, t);
     const int n_new = __ldcg(cu_seqlens + b + 1) - __ldcg(cu_seqlens + b);
@@ -58,7 +65,7 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         return 0.f;
     };
 #pragma unroll 2
-    for (int c = threadIdx.x; c < C; c += CI_THREADS) {
+    for (int c = c0 + threadIdx.x; c < c1; c += CI_THREADS) {
         const float bc = bias != nullptr ? to_f32(bias[c]) : 0.f;
         float acc;
         if (ntaps <= 0) {
@@ -99,7 +106,7 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
     if (norm_last && cs != nullptr) {
         // The pairs of every query and key head in place, a thread per pair.
         __syncthreads();
-        for (int e = threadIdx.x; e < (nq + (write_kv ? nkv : 0)) * half; e += CI_THREADS) {
+        for (int e = qk0 * half + threadIdx.x; e < qk1 * half; e += CI_THREADS) {
             const int i = e % half;
             float* src = y + (size_t)(e / half) * D;
             const int a = interleaved ? 2 * i : i, c = interleaved ? 2 * i + 1 : i + half;
@@ -113,8 +120,7 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         // A warp per head: the order of a head's sum depends on the head's size alone.
         __syncthreads();
         const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-        const int heads = nq + (write_kv ? nkv : 0);
-        for (int hd = warp; hd < heads; hd += CI_THREADS / 32) {
+        for (int hd = qk0 + warp; hd < qk1; hd += CI_THREADS / 32) {
             const T* w = hd < nq ? q_norm_w : k_norm_w;
             if (w == nullptr) continue;
             float* src = y + (size_t)hd * D;
@@ -129,14 +135,13 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
     if (q_norm_w != nullptr) invq = 1.0f / sqrtf(block_sum(ssq, scratch) / (float)Cq + eps);
     if (k_norm_w != nullptr && write_kv) invk = 1.0f / sqrtf(block_sum(ssk, scratch) / (float)Ck + eps);
     __syncthreads();
-    for (int c = threadIdx.x; c < Cq + Ck; c += CI_THREADS) {
+    for (int c = c0 + threadIdx.x; c < min(c1, Cq + Ck); c += CI_THREADS) {
         if (c < Cq) { if (q_norm_w != nullptr) y[c] = y[c] * invq * to_f32(q_norm_w[c]); }
         else if (k_norm_w != nullptr) y[c] = y[c] * invk * to_f32(k_norm_w[c - Cq]);
     }
     __syncthreads();
     // Queries and keys: heads of Dp elements, the first D from y (rotated where the rotation reaches), zeros after.
-    const int qk_heads = nq + (write_kv ? nkv : 0);
-    for (int e = threadIdx.x; e < qk_heads * Dp; e += CI_THREADS) {
+    for (int e = qk0 * Dp + threadIdx.x; e < qk1 * Dp; e += CI_THREADS) {
         const int head = e / Dp, d = e % Dp;
         float v = 0.f;
         if (d < D) {
@@ -152,7 +157,7 @@ __global__ void __launch_bounds__(CI_THREADS) conv_attention_inputs_kernel(
         else k_cache[(((size_t)page * nkv + head - nq) * page_size + off) * Dp + d] = from_f32<T>(v);
     }
     if (write_kv && !shared_kv)
-        for (int e = threadIdx.x; e < nkv * Dp; e += CI_THREADS) {
+        for (int e = v0 * Dp + threadIdx.x; e < v1 * Dp; e += CI_THREADS) {
             const int head = e / Dp, d = e % Dp;
             v_cache[(((size_t)page * nkv + head) * page_size + off) * Dp + d] = from_f32<T>(d < V ? y[Cq + Ck + head * V + d] : 0.f);
         }
@@ -179,10 +184,18 @@ extern "C" int ti_conv_attention_inputs(const void* proj, long long ld, const vo
     const int C = nq * D + (write_kv ? nkv * (shared_kv ? D : D + V) : 0);
     const size_t smem = (size_t)C * sizeof(float);
     TI_REQUIRE(smem <= 160 * 1024, "conv_attention_inputs: %d channels", C);
+    // Few tokens: their heads are shared out among several blocks each (a head's results do not depend on it).
+    int parts = 1;
+    if (!shared_kv && (head_norm || (q_norm_w == nullptr && k_norm_w == nullptr))) {
+        parts = 4 * ti_sm_count() / n;
+        if (parts > C / CI_THREADS) parts = C / CI_THREADS;
+        if (parts > nq) parts = nq;
+        if (parts < 1) parts = 1;
+    }
 #define CI_LAUNCH(TAPS)                                                                                                                       \
     do {                                                                                                                                      \
         if (smem > 48 * 1024) cudaFuncSetAttribute(conv_attention_inputs_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        ti_launch(conv_attention_inputs_kernel<T, TAPS>, dim3(n), dim3(CI_THREADS), smem, stream, (const T*)proj, ld, (const T*)bias, (const T*)conv,  \
+        ti_launch(conv_attention_inputs_kernel<T, TAPS>, dim3(n, parts), dim3(CI_THREADS), smem, stream, (const T*)proj, ld, (const T*)bias, (const T*)conv,  \
                   taps, state, (const T*)q_norm_w, (const T*)k_norm_w, eps, cos_sin, rotary, (T*)q_out, (T*)k_cache, (T*)v_cache, positions,       \
                   slot_map, cu_seqlens, seq_slots, kv_lens, B, nq, nkv, D, V, Dp, page_size, write_kv, head_norm, shared_kv, interleaved, norm_last);   \
     } while (0)

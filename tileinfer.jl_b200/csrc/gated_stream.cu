@@ -3,6 +3,8 @@
 //
 //   gated_add_norm32   x += mult * (d + bias) * sigmoid(g + gbias);  h = T(G(x) * w), G: the row in `groups` equal parts, each divided by
 //                      its own sqrt(mean(part^2) + eps) (`offset`: times 1 + w);  for one-token steps also hc = T(h + conv(h)) from and to the sequences' history
+//   pair_add_norm32    the same for two sublayers side by side, each normed over the row first:
+//                      x += mult * (sa A / rms(A) * wa + sb B / rms(B) * wb);  h = T(x / rms(x) * w)
 //   conv_rows          hc = T(h + conv(h)), conv(h)_t = sum_j c[j] * h_(t - taps + 1 + j) per channel, over a step's rows (rows before the
 //                      step from the history; its update is history_update, a launch of its own, since these blocks read it)
 //
@@ -203,6 +205,79 @@ extern "C" int ti_gated_add_norm32(float* x, const void* d, const float* d_parti
         else ti_launch(gated_add_norm32_kernel<T, 1>, dim3(n_rows), dim3(threads), smem, stream, x, db, gb, (T*)h, (const T*)w, eps, groups, cs, size, has_branch, has_gate, mult, offset);
     });
     return ti_check_launch("gated_add_norm32");
+}
+
+// ------------------------------------------------------------------------------------------------ two sublayers at once
+struct PairSum {
+    BranchRows a, b;
+    const void* wa;
+    const void* wb;
+    float sa, sb, eps;
+};
+template <typename T, int VEC>
+__global__ void pair_add_norm32_kernel(float* x, PairSum p, T* __restrict__ h, const T* __restrict__ w, float eps, float mult, int offset, int size) {
+    extern __shared__ __align__(16) float rows[];        // [2][size]: A and B, then the stream's new row
+    __shared__ float scratch[33];
+    const int row = blockIdx.x, padded = (size + 3) / 4 * 4;
+    float* xr = x + (size_t)row * size;
+    float ssa = 0.f, ssb = 0.f, ss = 0.f;
+    pdl_enter();
+    for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {
+        float va[VEC], vb[VEC];
+        branch_piece<T, VEC>(p.a, row, size, i, va);
+        branch_piece<T, VEC>(p.b, row, size, i, vb);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { ssa = fmaf(va[e], va[e], ssa); ssb = fmaf(vb[e], vb[e], ssb); }
+        Piece<float, VEC>::store(rows + i, va);
+        Piece<float, VEC>::store(rows + padded + i, vb);
+    }
+    const float ia = p.sa / sqrtf(block_sum(ssa, scratch) / (float)size + p.eps), ib = p.sb / sqrtf(block_sum(ssb, scratch) / (float)size + p.eps);
+    for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {       // (a thread reads back the elements it wrote)
+        float v[VEC], wa[VEC], wb[VEC];
+        Piece<float, VEC>::load(xr + i, v);
+        Piece<T, VEC>::load((const T*)p.wa + i, wa);
+        Piece<T, VEC>::load((const T*)p.wb + i, wb);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            v[e] = fmaf(mult, fmaf(rows[i + e] * ia, wa[e], rows[padded + i + e] * ib * wb[e]), v[e]);
+            ss = fmaf(v[e], v[e], ss);
+        }
+        Piece<float, VEC>::store(xr + i, v);
+        Piece<float, VEC>::store(rows + i, v);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)size + eps);
+    for (int i = threadIdx.x * VEC; i < size; i += blockDim.x * VEC) {
+        float v[VEC], wv[VEC];
+        Piece<T, VEC>::load(w + i, wv);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = rows[i + e] * inv * (offset ? 1.0f + wv[e] : wv[e]);
+        Piece<T, VEC>::store(h + (size_t)row * size + i, v);
+    }
+}
+
+// a, b: rows [n, size] with a stride, or partial sums with floats between parts, as ti_gated_add_norm32 takes them; wa, wb, w [size] of T.
+extern "C" int ti_pair_add_norm32(float* x, const void* a, const float* a_partials, int a_n, long long a_stride, const void* b, const float* b_partials, int b_n,
+                                  long long b_stride, const void* wa, const void* wb, float sa, float sb, float pair_eps, float mult, void* h, const void* w,
+                                  int offset, float eps, int n_rows, int size, int dtype, cudaStream_t stream) {
+    if (n_rows == 0) return 0;
+    TI_REQUIRE(size > 0 && size <= 20000, "pair_add_norm32: rows of %d", size);
+    TI_REQUIRE((a != nullptr) != (a_partials != nullptr) && (b != nullptr) != (b_partials != nullptr), "pair_add_norm32: each side is rows or partial sums");
+    TI_REQUIRE(wa != nullptr && wb != nullptr && w != nullptr && h != nullptr, "pair_add_norm32: the norms need their weights");
+    const PairSum p = {{a, a_partials, a_n, a_stride, nullptr, nullptr, 0, nullptr}, {b, b_partials, b_n, b_stride, nullptr, nullptr, 0, nullptr}, wa, wb, sa, sb, pair_eps};
+    const int threads = size >= 4096 ? 512 : size >= 1024 ? 256 : 128;
+    const size_t smem = (size_t)2 * ((size + 3) / 4 * 4) * sizeof(float);
+    TI_DISPATCH_DTYPE(dtype, {
+        const uintptr_t mask = sizeof(T) == 2 ? 7 : 15;
+        const bool vec = size % 4 == 0 && aligned16(x) && (((uintptr_t)h | (uintptr_t)w | (uintptr_t)wa | (uintptr_t)wb) & mask) == 0 && row_vec_ok(p.a, sizeof(T)) &&
+                         row_vec_ok(p.b, sizeof(T));
+        if (smem > 48 * 1024) {
+            cudaFuncSetAttribute(pair_add_norm32_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            cudaFuncSetAttribute(pair_add_norm32_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        }
+        if (vec) ti_launch(pair_add_norm32_kernel<T, 4>, dim3(n_rows), dim3(threads), smem, stream, x, p, (T*)h, (const T*)w, eps, mult, offset, size);
+        else ti_launch(pair_add_norm32_kernel<T, 1>, dim3(n_rows), dim3(threads), smem, stream, x, p, (T*)h, (const T*)w, eps, mult, offset, size);
+    });
+    return ti_check_launch("pair_add_norm32");
 }
 
 // ------------------------------------------------------------------------------------------------ the convolution over a step's rows

@@ -247,8 +247,9 @@ _SIGNATURES.update({
                         _I, _P],
 })
 
-# The state-space recurrence: inputs, one-token step, chunks of a prompt, gate and norm of its output.
+# The update of a stream by two sublayers side by side. The state-space recurrence: inputs, one-token step, chunks of a prompt, gate and norm of its output.
 _SIGNATURES.update({
+    "ti_pair_add_norm32": [_P, _P, _P, _I, _L, _P, _P, _I, _L, _P, _P, _F, _F, _F, _F, _P, _P, _I, _F, _I, _I, _I, _P],
     "ti_ssm_inputs": [_P, _P, _P, _L, _I, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "ti_ssm_token": [_P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "ti_ssm_chunks": [_P, _P, _L, _I, _I, _I, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],

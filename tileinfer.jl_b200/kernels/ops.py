@@ -768,6 +768,15 @@ def gated_add_norm32(x, d, gate, h, w, eps, groups=1, d_bias=None, gate_bias=Non
                                     n, size, dtype_code(h.dtype), _stream()), "gated_add_norm32")
 
 
+def pair_add_norm32(x, a, b, wa, wb, scale_a, scale_b, pair_eps, mult, h, w, eps, offset=False):
+    """x += mult * (scale_a A / rms(A) * wa + scale_b B / rms(B) * wb) on a 32-bit stream, then h = x / rms(x) * w (``offset``: times 1 + w).
+    A, B: rows [n, size] or 32-bit partial sums [s, n, size]."""
+    _need(x, "x", torch.float32); _need(h, "h"); _need(w, "w", h.dtype); _need(wa, "wa", h.dtype); _need(wb, "wb", h.dtype)
+    n, size = x.shape
+    check(lib().ti_pair_add_norm32(x.data_ptr(), *_branch_args(a, h.dtype, "a"), *_branch_args(b, h.dtype, "b"), wa.data_ptr(), wb.data_ptr(), scale_a, scale_b,
+                                   pair_eps, mult, h.data_ptr(), w.data_ptr(), int(bool(offset)), eps, n, size, dtype_code(h.dtype), _stream()), "pair_add_norm32")
+
+
 def conv_rows(out, h, conv, hist, step):
     """out = h + conv(h) over a step's rows, conv [taps, size] causal per channel, earlier rows from the sequences' history ``hist``
     [slots, >= (taps - 1) * size] float32 (None with one tap); ``history_update`` moves the history on afterwards."""

@@ -267,7 +267,7 @@ class GatedBlock(Part):
     The gates read h as the norm left it, before the convolution. Options: ``residual_mult`` m (default 1); ``taps`` (0: no convolution, the mixer reads h) with ``conv``
     the name of its weights [size, taps]; ``gates``: the names of R1 and R2 [size, size], whose biases have ``bias_suffix`` added (None:
     no gates). A mixer whose output projection has a bias (``out_bias``) leaves it to the kernel that updates the stream; a
-    routed feed-forward leaves a token's rows apart for it. The norms are of a kind that offers ``gated_add`` (``rmsnorm32``)."""
+    routed feed-forward leaves a token's rows apart for it, a pair of mixers its two outputs. The norms are of a kind that offers ``gated_add`` (``rmsnorm32``)."""
 
     def __init__(self, spec, mixer, feed_forward, mixer_norm, feed_forward_norm, tensors, rt):
         self.spec, self.rt = spec, rt
@@ -278,8 +278,9 @@ class GatedBlock(Part):
         self.taps = int(o.get("taps") or 0)
         # Kept [taps, size]: neighbouring channels' weights of one tap lie together.
         self.conv = rt.param(tensors[o["conv"]]).t().contiguous() if self.taps else None
-        if hasattr(feed_forward, "rows_apart"):
-            feed_forward.rows_apart = True
+        for part in (mixer, feed_forward):
+            if hasattr(part, "rows_apart"):
+                part.rows_apart = True
         self.gates, self.gate_biases = [], []
         for name in (o.get("gates") or ())[:2 if feed_forward is not None else 1]:
             gate = Linear(rt.param(tensors[name]), rt, "residual_gate")

@@ -3,6 +3,8 @@
 precedes it (src/ops/tile/norm.jl:48-77). No bias, no ``1 + w``."""
 from __future__ import annotations
 
+import torch
+
 from ..config.spec import NormSpec, TensorDecl
 from ..kernels import ops
 from .base import Norm, register_norm
@@ -70,10 +72,15 @@ class RMSNorm32(Norm):
 
     def gated_add(self, x, delta, out, gate=None, bias=None, gate_bias=None, conv=None, mult=1.0):
         """x += mult * (delta + bias) * sigmoid(gate + gate_bias) on a 32-bit stream (``delta`` None: x stays), then out = norm(x). ``delta``:
-        rows, 32-bit partial sums or :class:`GatheredRows` with weights; ``gate``: rows or partial sums, None for no gate. ``conv``: see
+        rows, 32-bit partial sums, :class:`GatheredRows` with weights or :class:`PairRows`; ``gate``: rows or partial sums, None for no gate. ``conv``: see
         ``ops.gated_add_norm32``."""
         if self.offset not in (False, True):
             raise NotImplementedError("a mean taken off is not built for gated_add")
+        if isinstance(delta, PairRows):
+            if gate is None and bias is None and conv is None and self.groups == 1:
+                ops.pair_add_norm32(x, delta.a, delta.b, delta.wa, delta.wb, delta.scale_a, delta.scale_b, delta.eps, mult, out, self.weight, self.eps, self.offset)
+                return out
+            delta = delta.combined(self.rt)
         common = dict(conv=conv, mult=mult, offset=self.offset)
         if isinstance(delta, GatheredRows):
             ops.gated_add_norm32(x, delta.rows, gate, out, self.weight, self.eps, self.groups, bias, gate_bias, delta.index, delta.scores, **common)
@@ -160,6 +167,21 @@ class GatheredRows:
 
     def __init__(self, rows, index, scores=None):
         self.rows, self.index, self.scores = rows, index, scores
+
+
+class PairRows:
+    """Two mixers' outputs that are still apart: their sum is scale_a a / rms(a) * wa + scale_b b / rms(b) * wb, every row normed over the
+    model's width. A norm that offers ``gated_add`` adds them up while it reads them. ``a``, ``b``: rows or 32-bit partial sums."""
+
+    def __init__(self, a, b, wa, wb, eps, scale_a, scale_b):
+        self.a, self.b, self.wa, self.wb, self.eps, self.scale_a, self.scale_b = a, b, wa, wb, eps, scale_a, scale_b
+
+    def combined(self, rt):
+        """The sum itself in 32-bit, shaped like one slice of partial sums."""
+        n, size = self.a.shape[-2:]
+        out = rt.buffer("pair.sum", (1, n, size), torch.float32)
+        ops.pair_combine(out[0], self.a, self.b, self.wa, self.wb, self.eps, self.scale_a, self.scale_b, rt.dtype)
+        return out
 
 
 class StreamCast(Norm):

@@ -15,6 +15,7 @@ import torch
 from ..config.spec import MixerSpec, TensorDecl
 from ..kernels import ops
 from .base import Mixer, lookup, register_mixer
+from .norm import PairRows
 
 
 @register_mixer("pair")
@@ -34,6 +35,8 @@ class MixerPair(Mixer):
         self.left_scale, self.right_scale = float(o.get("left_scale", 1.0)), float(o.get("right_scale", 1.0))
         self.out_norm = bool(o.get("out_norm", False))
         self.eps = float(o.get("norm_eps", 1e-6))
+        # Set by a block whose stream update norms and adds the two outputs itself: they then come as PairRows.
+        self.rows_apart = False
         n, p = spec.tensor_names, spec.prefix
         self.w_left = rt.param(tensors[p + n["left_out"]]) if self.out_norm else None
         self.w_right = rt.param(tensors[p + n["right_out"]]) if self.out_norm else None
@@ -61,6 +64,8 @@ class MixerPair(Mixer):
     def forward(self, h, step, cache):
         a = self.left.forward(h, step, cache)
         b = self.right.forward(h, step, cache)
+        if self.rows_apart and self.out_norm:
+            return PairRows(a, b, self.w_left, self.w_right, self.eps, self.left_scale, self.right_scale)
         out = self.rt.buffer("pair.sum", (1, h.shape[0], self.spec.hidden_size), torch.float32)
         ops.pair_combine(out[0], a, b, self.w_left, self.w_right, self.eps, self.left_scale, self.right_scale, self.rt.dtype)
         return out                                # 32-bit, shaped like one slice of partial sums: the stream's update adds it as it is
